@@ -52,6 +52,15 @@ class PagedKeysValues(CacheNeed):
                                            # later row, and the pages that hold them are never given back
 
 
+def span_covering(a: int, b: int) -> int:
+    """A span (`PagedKeysValues.window`) under which no page is given back that a row under span `a` or one under span `b` may
+    still read: either where they are equal, everything if one of them is everything, else a window of the larger size (a
+    row's own chunk of c positions begins at most c - 1 positions in front of it)."""
+    if a == b:
+        return a
+    return 0 if a == 0 or b == 0 else max(abs(a), abs(b))
+
+
 @dataclass(frozen=True)
 class FixedState(CacheNeed):
     shape: Tuple[int, ...]

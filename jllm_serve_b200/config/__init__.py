@@ -1,6 +1,6 @@
 """Typed configuration and the architecture registry."""
 from .specs import (AttentionNames, ConfigError, Core, Decoder, DenseGluSpec, DenseMlpSpec, FeedForwardSpec, MatrixMemorySpec,
-                    SelectiveStateSpaceSpec, FixedDecayLinearAttentionSpec,
+                    SelectiveStateSpaceSpec, FixedDecayLinearAttentionSpec, GeneralDeltaSpec,
                     GatedLinearAttentionSpec, GqaAttentionSpec, LatentAttentionSpec, LayerNames, LayerRun, LayerSpec, ModelNames,
                     MixerSpec, NormSpec, ParallelMixersSpec, RopeScaling, RopeTableSpec, RoutedExpertsSpec)
 from .reader import ConfigReader
@@ -11,9 +11,11 @@ from .madevik import parse_madevik
 from .movivik import parse_movivik
 from .bozevik import parse_bozevik
 from .guvolix import parse_guvolix
+from .fusazen import parse_fusazen
 
 register_architecture("qwen3", parse_qwen3, replace=True)
 register_architecture("Madevik", parse_madevik, replace=True)
 register_architecture("Movivik", parse_movivik, replace=True)
 register_architecture("Bozevik", parse_bozevik, replace=True)
 register_architecture("Guvolix", parse_guvolix, replace=True)
+register_architecture("Fusazen", parse_fusazen, replace=True)

@@ -87,6 +87,8 @@ class AttentionNames:
     k_norm: str = "k_norm.weight"
     gate: str = "gate.weight"
     sink: str = "sink"
+    head_scale: str = "head_scale"
+    lambdas: Tuple[str, str, str, str] = ("lambda_q1", "lambda_k1", "lambda_q2", "lambda_k2")
 
 
 @dataclass(frozen=True)
@@ -94,7 +96,12 @@ class GqaAttentionSpec(MixerSpec):
     """Grouped-query causal attention over a paged cache (Attention.java:48-50,68-71). Beyond the reference's: value heads
     of another width than key heads (`value_dim`), rows that see only their own chunk of the sequence (`chunk`), a division
     of every query and key head by its root mean square behind the rotation (`unit_qk`), and a sigmoid gate per head on the
-    attention's result, read from the mixer's input by one more projection (`gate`)."""
+    attention's result, read from the mixer's input by one more projection (`gate`); a norm over ALL rows of the query (key)
+    projection at once (`qk_norm_over` = "all"), a learned factor per query head on the scores (`head_scale`); and a differential
+    attention (`maps` = 2): every head's query and key are two maps [map 1, map 2] of head_dim values each, both attend the same
+    values, and with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff the head's result is rms(a1 - lambda a2) (1 - diff). A
+    mixer with `own_kv` False has no key and value projections: it reads the rows that another run cached (the schedule's
+    `cache_of`), with its own queries and mask."""
     kind: str = field(default="gqa_attention", init=False)
     heads: int = 0
     kv_heads: int = 0
@@ -114,6 +121,13 @@ class GqaAttentionSpec(MixerSpec):
     names: AttentionNames = AttentionNames()
     keep_first: int = 0                    # with a window: the sequence's first keep_first positions stay visible to every row
     sink: bool = False                     # a learned number per query head whose exponential joins the softmax's denominator
+    qk_norm_over: str = "head"             # head: one gain of head_dim values for every head | all: the rows of q (of k) are
+                                           # normed together, with a gain of that many values
+    head_scale: bool = False               # scores also times a stored number per query head
+    maps: int = 1                          # 2: differential attention
+    diff: float = 0.0                      # its constant
+    diff_norm_eps: float = 1e-6            # eps of the norm over a head's difference
+    own_kv: bool = True                    # False: no key and value projections, another run's cache
 
     def __post_init__(self):
         if self.heads <= 0:
@@ -133,10 +147,33 @@ class GqaAttentionSpec(MixerSpec):
             raise ConfigError(f"attention: gate {self.gate!r} is not built (built: none, head_sigmoid, sigmoid)")
         if self.keep_first < 0 or (self.keep_first and not self.window):
             raise ConfigError(f"attention: keep_first={self.keep_first} must not be negative and needs a window")
+        if self.qk_norm_over not in ("head", "all") or self.maps not in (1, 2):
+            raise ConfigError(f"attention: qk_norm_over={self.qk_norm_over!r} maps={self.maps} is not built")
+        if self.wide and (self.bias or self.out_bias or self.gate != "none" or self.sink or self.unit_qk
+                          or (self.qk_norm and self.qk_norm_over == "head")):
+            raise ConfigError("attention: two maps per head, norms over all heads and a factor per head are not built together "
+                              "with biases, gates, sinks, unit queries or norms per head")
 
     @property
     def v_dim(self) -> int:
         return self.value_dim or self.head_dim
+
+    @property
+    def wide(self) -> bool:
+        """Whether the rows are prepared by the kernel that lays a head's maps side by side in rows of `row_dim` values."""
+        return self.maps > 1 or self.head_scale or not self.own_kv or (self.qk_norm and self.qk_norm_over == "all")
+
+    @property
+    def row_dim(self) -> int:
+        """Values of a cached row. A wide attention's key row holds the head's maps side by side and its value row the value,
+        both filled up with zeros to a width that the tile kernels take where at most a third is added to get there."""
+        if not self.wide:
+            return max(self.head_dim, self.v_dim)
+        w = max(self.maps * self.head_dim, self.v_dim)
+        for tile in (64, 128, 256):
+            if w <= tile <= w + w // 3:
+                return tile
+        return -(-w // 16) * 16 if w <= 256 else -(-w // 8) * 8
 
 
 @dataclass(frozen=True)
@@ -161,6 +198,33 @@ class GatedLinearAttentionSpec(MixerSpec):
             raise ConfigError(f"gated linear attention: decay_rank={self.decay_rank} must be positive (or -1: as stored)")
         if not self.decay_temperature > 0:
             raise ConfigError(f"gated linear attention: tau={self.decay_temperature} must be positive")
+
+
+@dataclass(frozen=True)
+class GeneralDeltaSpec(MixerSpec):
+    """A recurrence whose transition is a decay per key channel minus a rank-one removal (a generalized delta rule): r, k, v =
+    Wr h, Wk h, Wv h; d = exp(-decay_rate sigmoid(W2 tanh(W1 h) + w0)) and a = sigmoid(Wa h + ba) per head and key channel; with
+    the unit key u = k / sqrt(sum(k^2) + 1e-6) of a head S_t = diag(d_t) S_(t-1) - (a_t u_t) (u_t^T S_(t-1)) + k_t v_t^T,
+    o_t = S_t^T r_t; each head's o over its root mean square, a gain over all heads, a sigmoid gate of full width, the output
+    projection. State per request: S [heads, key_dim, value_dim], float32."""
+    kind: str = field(default="general_delta", init=False)
+    heads: int = 0
+    key_dim: int = 0
+    value_dim: int = 0
+    decay_rate: float = 0.6065306597126334     # exp(-1/2): the largest decay of a token is exp(-decay_rate)
+    decay_rank: int = -1                       # width of the low-rank decay projection (rows of W1); -1: the checkpoint's own
+    norm_eps: float = 1e-6
+
+    def __post_init__(self):
+        for name in ("heads", "key_dim", "value_dim"):
+            if getattr(self, name) <= 0:
+                raise ConfigError(f"delta rule: {name}={getattr(self, name)} must be positive")
+        if self.decay_rank == 0 or self.decay_rank < -1:
+            raise ConfigError(f"delta rule: decay_rank={self.decay_rank} must be positive (or -1: as stored)")
+        if not self.decay_rate > 0:
+            raise ConfigError(f"delta rule: decay_rate={self.decay_rate} must be positive")
+        if self.key_dim > 1024:
+            raise ConfigError(f"delta rule: dim={self.key_dim} (built: up to 1024)")
 
 
 @dataclass(frozen=True)
@@ -350,17 +414,20 @@ class DenseGluSpec(FeedForwardSpec):
 
 @dataclass(frozen=True)
 class DenseMlpSpec(FeedForwardSpec):
-    """down(act(up x)): two matrices and no gate."""
+    """down(act(up x)): two matrices and no gate, with or without biases."""
     kind: str = field(default="dense_mlp", init=False)
     hidden: int = 0
-    activation: str = "gelu_erf"           # gelu_erf: z (1 + erf(z / sqrt 2)) / 2
+    activation: str = "gelu_erf"           # gelu_erf: z (1 + erf(z / sqrt 2)) / 2 | relu2: max(z, 0)^2
     names: Tuple[str, str] = ("up", "down")
+    bias_names: Tuple[str, ...] = ()       # empty: no biases; else the names of the two products' biases
 
     def __post_init__(self):
         if self.hidden <= 0:
             raise ConfigError(f"feed-forward: ff={self.hidden} must be positive")
-        if self.activation not in ("gelu_erf",):
-            raise ConfigError(f"unsupported activation {self.activation!r} of an ungated feed-forward (built: gelu_erf)")
+        if self.activation not in ("gelu_erf", "relu2"):
+            raise ConfigError(f"unsupported activation {self.activation!r} of an ungated feed-forward (built: gelu_erf, relu2)")
+        if len(self.bias_names) not in (0, 2):
+            raise ConfigError("feed-forward: biases are named for both products or for none")
 
 
 @dataclass(frozen=True)
@@ -445,6 +512,10 @@ class LayerSpec:
     prefix: Optional[str] = None           # the layer's checkpoint prefix where it is not ModelNames.layer.format(index)
     token_shift: str = ""                  # "": none; else the name (under the layer's prefix) of a vector mu: the mixer
                                            # reads x_t + (x_(t-1) - x_t) * mu, x_(-1) = 0 (`post_norm` arrangement)
+    input_conv: str = ""                   # "": none; else the name (under the layer's prefix) of a table c [width, taps]: the
+                                           # mixer reads h_t + sum_j c[:, j] h_(t - taps + 1 + j), h the normed rows, zeros in
+                                           # front of the sequence (`pre_norm` arrangement)
+    input_conv_taps: int = 0
 
 
 @dataclass(frozen=True)

@@ -191,6 +191,15 @@ __device__ __forceinline__ float glu_unit(float gate, float up, int word) {
     return __fmul_rn(glu_act<FAST>(gate, word), up);
 }
 
+// What a product does with its result, the launchers' `accumulate` argument: 0 store it, 1 add it to what `out` holds, 2
+// store max(v, 0)^2 (the activation of an ungated feed-forward; behind the bias).
+enum : int { EPI_STORE = 0, EPI_ADD = 1, EPI_RELU2 = 2 };
+__device__ __forceinline__ float epilogue_act(float v, int how) {
+    if (how != EPI_RELU2) return v;
+    const float z = fmaxf(v, 0.f);
+    return __fmul_rn(z, z);
+}
+
 // A vector (gain, bias) whose stored type is known only at run time.
 struct VecRef {
     const void* p;

@@ -64,7 +64,7 @@ struct TileEpilogue {
     // All 32 rows of the warp lie inside the matrix and float32 rows can be accessed 16 bytes at a time: the block goes
     // through shared memory (`staged`).
     __device__ __forceinline__ bool rows_whole(int row0) const {
-        return !swiglu && row0 + 32 <= M && sizeof(Tout) == 4 && (ldo & 3) == 0 && (((uintptr_t)out) & 15u) == 0;
+        return !swiglu && accumulate != EPI_RELU2 && row0 + 32 <= M && sizeof(Tout) == 4 && (ldo & 3) == 0 && (((uintptr_t)out) & 15u) == 0;
     }
 
     // Through shared memory, so that a warp's accesses are whole lines: a thread holds 32 values of ONE row, and
@@ -152,15 +152,19 @@ struct TileEpilogue {
                             r.z += bias[n_base + 4 * j + 2];
                             r.w += bias[n_base + 4 * j + 3];
                         }
+                        r.x = epilogue_act(r.x, accumulate);
+                        r.y = epilogue_act(r.y, accumulate);
+                        r.z = epilogue_act(r.z, accumulate);
+                        r.w = epilogue_act(r.w, accumulate);
                         if (vec) {
-                            if (accumulate) {
+                            if (accumulate == EPI_ADD) {
                                 const float4 o = d4[j];
                                 r.x += o.x; r.y += o.y; r.z += o.z; r.w += o.w;
                             }
                             d4[j] = r;
                         } else {
                             float* d = reinterpret_cast<float*>(dst) + 4 * j;
-                            if (accumulate) { r.x += d[0]; r.y += d[1]; r.z += d[2]; r.w += d[3]; }
+                            if (accumulate == EPI_ADD) { r.x += d[0]; r.y += d[1]; r.z += d[2]; r.w += d[3]; }
                             d[0] = r.x; d[1] = r.y; d[2] = r.z; d[3] = r.w;
                         }
                     }
@@ -173,7 +177,9 @@ struct TileEpilogue {
                         for (int e = 0; e < 4; ++e) {
                             float lo = __uint_as_float(v[8 * j + 2 * e]), hi = __uint_as_float(v[8 * j + 2 * e + 1]);
                             if (has_bias) { lo += bias[n_base + 8 * j + 2 * e]; hi += bias[n_base + 8 * j + 2 * e + 1]; }
-                            if (accumulate) { lo += to_float(dst[8 * j + 2 * e]); hi += to_float(dst[8 * j + 2 * e + 1]); }
+                            lo = epilogue_act(lo, accumulate);
+                            hi = epilogue_act(hi, accumulate);
+                            if (accumulate == EPI_ADD) { lo += to_float(dst[8 * j + 2 * e]); hi += to_float(dst[8 * j + 2 * e + 1]); }
                             __nv_bfloat162 b2 = __floats2bfloat162_rn(lo, hi);
                             p[e] = *reinterpret_cast<uint32_t*>(&b2);
                         }
@@ -195,7 +201,8 @@ struct TileEpilogue {
                     if (n_base + j < N) {
                         float r = __uint_as_float(v[j]);
                         if (has_bias) r += bias[n_base + j];
-                        if (accumulate) r += to_float(dst[j]);
+                        r = epilogue_act(r, accumulate);
+                        if (accumulate == EPI_ADD) r += to_float(dst[j]);
                         dst[j] = from_float<Tout>(r);
                     }
                 }

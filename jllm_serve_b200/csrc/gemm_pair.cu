@@ -490,7 +490,7 @@ JLLM_EXPORT int jllm_gemm_pair(const void* a, int lda, const void* w, int k_bloc
     rc = packed_map_for(w, packed_rows, &map_w);
     if (rc != JLLM_OK) return rc;
     CUtensorMap map_out = {};
-    const int bulk_out = out_dtype == JLLM_F32 && !swiglu && ldo % 4 == 0 && ((uintptr_t)out % 16) == 0 && !g_plain_stores;
+    const int bulk_out = out_dtype == JLLM_F32 && !swiglu && accumulate != EPI_RELU2 && ldo % 4 == 0 && ((uintptr_t)out % 16) == 0 && !g_plain_stores;
     if (bulk_out) {
         rc = tensor_map_out_f32(out, M, N, ldo, &map_out);
         if (rc != JLLM_OK) return rc;

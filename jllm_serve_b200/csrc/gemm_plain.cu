@@ -56,7 +56,8 @@ gemm_plain_kernel(const Tin* __restrict__ a, int lda, const Tin* __restrict__ w,
             float v = acc[i][j];
             if (has_bias) v += bias[n];
             Tout* dst = out + (size_t)m * ldo + n;
-            if (accumulate) v += to_float(*dst);
+            v = epilogue_act(v, accumulate);
+            if (accumulate == EPI_ADD) v += to_float(*dst);
             *dst = from_float<Tout>(v);
         }
     }

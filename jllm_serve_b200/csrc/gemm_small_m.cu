@@ -173,7 +173,8 @@ gemm_small_m_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfl
         }
         if (has_bias) v += bias[n];
         Tout* dst = out + (size_t)tok * ldo + n;
-        if (accumulate) v += to_float(*dst);
+        v = epilogue_act(v, accumulate);
+        if (accumulate == EPI_ADD) v += to_float(*dst);
         *dst = from_float<Tout>(v);
     }
 }

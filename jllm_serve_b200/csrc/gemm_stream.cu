@@ -195,10 +195,10 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_a, const __nv_bfloat1
                     // all the old values are requested before the first store (a load behind a store through the
                     // same pointer would wait for it: 16 round trips instead of one)
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) old[j] = (accumulate && m0 + j < M) ? to_float(dst[(size_t)j * ldo]) : 0.f;
+                    for (int j = 0; j < 16; ++j) old[j] = (accumulate == EPI_ADD && m0 + j < M) ? to_float(dst[(size_t)j * ldo]) : 0.f;
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
-                        if (m0 + j < M) dst[(size_t)j * ldo] = from_float<Tout>((v[j] + b) + old[j]);
+                        if (m0 + j < M) dst[(size_t)j * ldo] = from_float<Tout>(epilogue_act(v[j] + b, accumulate) + old[j]);
                 }
             };
             if (kb0 == 0 && kb1 == k_blocks) {                      // the whole tile is this block's

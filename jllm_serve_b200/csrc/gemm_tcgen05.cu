@@ -401,7 +401,7 @@ JLLM_EXPORT int jllm_gemm_tcgen05(const void* a, int lda, const void* w, int k_b
     if (rc != JLLM_OK) return rc;
     // a float32 output leaves by tiled bulk copies (the residual add as a reduce in L2) where its rows allow a tensor map
     CUtensorMap map_out = {};
-    const int bulk_out = out_dtype == JLLM_F32 && !swiglu && ldo % 4 == 0 && ((uintptr_t)out % 16) == 0 && !g_plain_stores;
+    const int bulk_out = out_dtype == JLLM_F32 && !swiglu && accumulate != EPI_RELU2 && ldo % 4 == 0 && ((uintptr_t)out % 16) == 0 && !g_plain_stores;
     if (bulk_out) {
         rc = tensor_map_out_f32(out, M, N, ldo, &map_out);
         if (rc != JLLM_OK) return rc;

@@ -192,6 +192,14 @@ class _Signatures:
     jllm_sigmoid_gate = [P, I, P, I, I, I, I, F, P]
     jllm_activation = [P, I, ctypes.c_longlong, I, P]
     jllm_add_rows_scaled = [P, P, I, I, P, I, I, I, P]
+    jllm_norm_conv = [P, P, I, P, I, P, I, P, P, P, P, P, I, I, I, I, I, F, I, P]
+    jllm_bounds_error_attention_maps = [P]
+    jllm_map_prepare = [P, I, I, I, I, P, P, F, P, P, I, I, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, P]
+    jllm_map_difference = [P, I, I, I, F, F, F, P, I, I, I, I, P]
+    jllm_bounds_error_delta_recurrence = [P]
+    jllm_delta_tanh = [P, I, P, I, I, I, P]
+    jllm_delta_recurrent = [P, I, I, I, I, I, P, P, I, F, P, I, P, P, P, P, I, I, I, I, P]
+    jllm_delta_chunked = [P, I, I, I, I, I, P, P, I, F, P, I, P, P, P, P, P, P, P, I, I, I, I, I, P]
     jllm_sample = [P, I, I, I, P, P, P, P, P, P, P]
 
 
@@ -400,6 +408,22 @@ def token_shift(x, mu, state, batch, out) -> None:
     _call("jllm_token_shift", x.data_ptr(), mu.data_ptr(), _DT[mu.dtype], state.data_ptr(), state.shape[0],
           batch.row_seg.data_ptr(), batch.seg_start.data_ptr(), batch.seg_len.data_ptr(), batch.state_slots.data_ptr(),
           out.data_ptr(), _DT[out.dtype], x.shape[0], batch.seg_start.numel(), x.shape[1], int(single), _stream())
+
+
+def norm_conv(x, gain, eps, conv, state, batch, out) -> None:
+    """out[r] = h_t + sum_j conv[:, j] h_(t - taps + 1 + j) with h = rmsnorm(x) * gain, within a segment; the rows in front of a
+    segment's first come from the request's state [slots, max(taps - 1, 1), dim] (its last taps - 1 normed rows, float32), which is
+    then brought up to date (a second launch unless every segment is one row). x float32 [rows, dim]; conv [dim, taps]."""
+    dim, taps = conv.shape
+    assert x.dtype == state.dtype == torch.float32 and x.is_contiguous() and state.is_contiguous() and out.is_contiguous()
+    assert conv.is_contiguous() and x.shape[1] == out.shape[1] == dim and tuple(state.shape[1:]) == (max(taps - 1, 1), dim)
+    single = batch.decode_only
+    global launch_count
+    launch_count += 0 if single or taps == 1 else 1
+    _call("jllm_norm_conv", x.data_ptr(), gain.data_ptr(), _DT[gain.dtype], conv.data_ptr(), _DT[conv.dtype], state.data_ptr(),
+          state.shape[0], batch.row_seg.data_ptr(), batch.seg_start.data_ptr(), batch.seg_len.data_ptr(),
+          batch.state_slots.data_ptr(), out.data_ptr(), _DT[out.dtype], x.shape[0], batch.seg_start.numel(), dim, taps, float(eps),
+          int(single), _stream())
 
 
 def depth_mix(stack, weights, n, out) -> None:
@@ -625,6 +649,77 @@ def head_prepare(qkv, q_off, k_off, v_off, q_gain, k_gain, eps, cos, sin, rotary
           int(write_kv), qkv.shape[0], heads, kv_heads, key_dim, value_dim, cache_dim, page_size, _stream())
 
 
+def map_prepare(src, k_off, v_off, q_gain, k_gain, eps, cos, sin, rotary_dim, pairing, positions, slots, q_out, k_cache, v_cache,
+                heads, kv_heads, maps, dim, value_dim, width, page_size, write_kv=True) -> None:
+    """The rows of a wide attention (see attention_maps.cu) from the stacked projection `src` [rows, *] (queries at column 0): an
+    optional RMS norm over all query (key) columns of a row with float32 gains per column; the rotation of the first `rotary_dim`
+    values of every map; query (head, map) to its own `width` values of q_out with zeros around it, the maps of a key head side by
+    side into one cache row, the value into another, zeros behind both. `write_kv` False: queries only."""
+    assert src.stride(1) == 1 and q_out.dtype == src.dtype and q_out.stride(1) == 1
+    assert all(g is None or (g.dtype == torch.float32 and g.is_contiguous()) for g in (q_gain, k_gain))
+    _call("jllm_map_prepare", src.data_ptr(), _DT[src.dtype], src.stride(0), int(k_off), int(v_off), _p(q_gain), _p(k_gain),
+          float(eps), _p(cos), _p(sin), int(rotary_dim), {"half": 0, "interleaved": 1}[pairing], positions.data_ptr(), _p(slots),
+          q_out.data_ptr(), q_out.stride(0), _p(k_cache), _p(v_cache), int(write_kv), src.shape[0], heads, kv_heads, maps, dim,
+          value_dim, width, page_size, _stream())
+
+
+def map_difference(att, width, lam, eps, out_scale, out, heads, value_dim) -> None:
+    """out[r, h] = rms(att[r, h, map 1] - lam * att[r, h, map 2]) * out_scale over a head's value_dim values; att [rows, heads x 2 x
+    width], out [rows, heads x value_dim]."""
+    assert att.dtype == out.dtype and att.stride(1) == 1 and out.stride(1) == 1
+    _call("jllm_map_difference", att.data_ptr(), _DT[att.dtype], att.stride(0), int(width), float(lam), float(eps), float(out_scale),
+          out.data_ptr(), out.stride(0), att.shape[0], heads, value_dim, _stream())
+
+
+def delta_tanh(src, out) -> None:
+    """out = tanh(src); src a float32 view [rows, width] with any row stride, out contiguous."""
+    assert src.dtype == torch.float32 and src.stride(1) == 1 and out.is_contiguous() and out.shape == src.shape
+    _call("jllm_delta_tanh", src.data_ptr(), src.stride(0), out.data_ptr(), _DT[out.dtype], src.shape[0], src.shape[1], _stream())
+
+
+def _delta_args(proj, r_off, k_off, v_off, a_off, z, a_bias, rate, state, seg_start, seg_len, state_slots, out):
+    assert proj.dtype == z.dtype == state.dtype == out.dtype == torch.float32 and proj.stride(1) == 1
+    assert z.is_contiguous() and state.is_contiguous() and out.is_contiguous()
+    return (proj.data_ptr(), proj.stride(0), int(r_off), int(k_off), int(v_off), int(a_off), z.data_ptr(), a_bias.data_ptr(),
+            _DT[a_bias.dtype], float(rate), state.data_ptr(), state.shape[0], seg_start.data_ptr(), seg_len.data_ptr(),
+            state_slots.data_ptr(), out.data_ptr())
+
+
+def delta_recurrent(proj, r_off, k_off, v_off, a_off, z, a_bias, rate, state, seg_start, seg_len, state_slots, out, heads, key_dim,
+                    value_dim) -> None:
+    """The generalized delta rule token by token: per (segment, head), with u = k / sqrt(sum(k^2) + 1e-6), d = exp(-rate
+    sigmoid(z)), a = sigmoid(a_raw + a_bias): S = diag(d) S - (a u) (u^T S) + k v^T, o = S^T r. proj float32 [rows, *]: r, k, a_raw
+    (heads x key_dim) and v (heads x value_dim) at the given columns; z float32 [rows, heads x key_dim]; state [slots, heads,
+    key_dim, value_dim] float32, read and written in place; out float32 [rows, heads x value_dim]."""
+    _call("jllm_delta_recurrent", *_delta_args(proj, r_off, k_off, v_off, a_off, z, a_bias, rate, state, seg_start, seg_len,
+                                               state_slots, out), seg_start.numel(), heads, key_dim, value_dim, _stream())
+
+
+DELTA_CHUNK = 32      # tokens of a chunk (C in delta_recurrence.cu)
+
+
+def delta_chunked(proj, r_off, k_off, v_off, a_off, z, a_bias, rate, state, seg_start, seg_len, state_slots, out, heads, key_dim,
+                  value_dim, max_len, qp, transition, added) -> bool:
+    """`delta_recurrent` for prompt portions, in chunks of 32 tokens (all float32; only the grouping of sums differs): three
+    launches. `max_len`: the longest segment's rows. qp [rows, heads x key_dim], transition [chunks, heads x key_dim x key_dim] and
+    added [chunks, heads x key_dim x value_dim] float32 scratch, chunks >= rows / 32 + segments. Says False, having launched
+    nothing, where the sizes are not taken."""
+    S = seg_start.numel()
+    assert qp.dtype == transition.dtype == added.dtype == torch.float32 and qp.is_contiguous()
+    if proj.shape[0] // DELTA_CHUNK + S > transition.shape[0]:
+        return False
+    code = library().jllm_delta_chunked(*_delta_args(proj, r_off, k_off, v_off, a_off, z, a_bias, rate, state, seg_start, seg_len,
+                                                     state_slots, out), qp.data_ptr(), transition.data_ptr(), added.data_ptr(), S,
+                                        int(max_len), heads, key_dim, value_dim, _stream())
+    if code == 3:        # the library's word for "these sizes are not taken"
+        return False
+    if code != 0:
+        raise KernelError(f"jllm_delta_chunked failed ({code}): {library().jllm_last_error().decode(errors='replace')}")
+    global launch_count
+    launch_count += 3
+    return True
+
+
 def head_gate(att, gate, heads, value_dim) -> None:
     """att[r, h, :] *= sigmoid(gate[r, h]) in place; att [rows, heads x value_dim], gate a view [rows, heads]."""
     assert att.dtype == gate.dtype and att.stride(1) == 1 and gate.stride(1) == 1 and att.shape[1] == heads * value_dim
@@ -648,6 +743,9 @@ def qk_norm_rope_store(qkv, q_gain, k_gain, eps, cos, sin, rotary_dim, positions
           _DT[q_gain.dtype] if use_norm else F32, int(use_norm), float(eps), _p(cos), _p(sin), int(rotary_dim),
           positions.data_ptr(), _p(slots), _p(k_cache), _p(v_cache), int(write_kv), qkv.shape[0], qkv.stride(0),
           heads, kv_heads, head_dim, page_size, _stream())
+
+
+EPILOGUE_RELU2 = 2       # as a product's `accumulate`: neither stored as it is (False) nor added (True), but max(v, 0)^2 stored
 
 
 def gemm_plain(a, w, out, bias=None, accumulate=False) -> None:
@@ -922,7 +1020,7 @@ def gemm_stream(a, packed: PackedWeight, out, bias=None, accumulate=False, swigl
 
 BOUNDS_FILES = ("attention_plain", "attention_decode", "attention_prefill", "attention_prefill_tc",
                 "attention_prefill_pair", "rowwise", "linear_attention", "latent_attention", "residual_paths",
-                "gated_recurrence")
+                "gated_recurrence", "attention_maps", "delta_recurrence")
 BOUNDS_WHAT = {1: "a block-table index", 2: "a page id", 3: "a cache slot", 4: "a token id", 5: "a row"}
 
 

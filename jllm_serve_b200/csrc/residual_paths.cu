@@ -16,6 +16,14 @@
 //                    plane behind it, and its blend with the next layer's saved row leaves in the compute type
 //   scale_values     x *= s
 //
+// and in front of a part whose input is blended over time:
+//   norm_conv        h = rms(x) * w;  out[r] = h_t + sum_j c[:, j] h_(t - taps + 1 + j) per channel: the layer's norm and a short
+//                    causal convolution over the normed rows in one launch. Rows in front of a segment's first come from the
+//                    request's state [slots, taps - 1, dim] (its last taps - 1 normed rows, float32, zeros for a new request),
+//                    which is brought up to date by the same launch when every segment is one row, else by
+//                    `norm_conv_save` behind it. A block takes eight neighbouring rows, so a row is normed once (and the
+//                    taps - 1 rows in front of the block once more).
+//
 // All arithmetic is float32; a row's result depends on that row (and the one in front of it) alone.
 #include "common.cuh"
 
@@ -270,6 +278,140 @@ __global__ void scale_values_kernel(float* __restrict__ x, float s, size_t count
         x[i] = __fmul_rn(x[i], s);
 }
 
+// The rms factors of the rows [lo, hi) into `inv` (a warp per row).
+__device__ __forceinline__ void rms_factors(const float* __restrict__ x, int lo, int hi, int dim, float eps, float* inv) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    for (int r = lo + warp; r < hi; r += warps) {
+        const float* src = x + (size_t)r * dim;
+        float ss = 0.f;
+        if ((dim & 3) == 0 && (((uintptr_t)x) & 15u) == 0) {
+            for (int i = lane * 4; i < dim; i += 128) {
+                const float4 v = *reinterpret_cast<const float4*>(src + i);
+                ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+            }
+        } else {
+            for (int i = lane; i < dim; i += 32) ss = fmaf(src[i], src[i], ss);
+        }
+        ss = warp_sum(ss);
+        if (lane == 0) inv[r - lo] = 1.f / sqrtf(ss / (float)dim + eps);
+    }
+}
+
+template <int V> struct Pack { float v[V]; };
+template <int V> __device__ __forceinline__ Pack<V> load_pack(const float* p) {
+    Pack<V> o;
+    if constexpr (V == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(p);
+        o.v[0] = x.x; o.v[1] = x.y; o.v[2] = x.z; o.v[3] = x.w;
+    } else {
+        o.v[0] = p[0];
+    }
+    return o;
+}
+template <int V> __device__ __forceinline__ void store_pack(float* p, const Pack<V>& o) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(o.v[0], o.v[1], o.v[2], o.v[3]);
+    else p[0] = o.v[0];
+}
+template <int V> __device__ __forceinline__ void store_pack(__nv_bfloat16* p, const Pack<V>& o) {
+    if constexpr (V == 4) {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(o.v[0], o.v[1]), hi = __floats2bfloat162_rn(o.v[2], o.v[3]);
+        uint2 u;
+        u.x = *reinterpret_cast<const uint32_t*>(&lo);
+        u.y = *reinterpret_cast<const uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>(p) = u;
+    } else {
+        p[0] = __float2bfloat16_rn(o.v[0]);
+    }
+}
+
+constexpr int CONV_TAPS = 16;     // most taps
+constexpr int CONV_RUN = 8;       // rows of a block in a step with prompt portions
+
+// RUN rows a block; `single` (RUN = 1): every segment is one row, and the state is brought up to date here. V channels a thread
+// at a time.
+template <typename Tout, int RUN, int V>
+__global__ void __launch_bounds__(256)
+norm_conv_kernel(const float* __restrict__ x, VecRef gain, VecRef conv, float* __restrict__ state, int num_slots,
+                 const int* __restrict__ row_seg, const int* __restrict__ seg_start, const int* __restrict__ state_slots,
+                 Tout* __restrict__ out, int rows, int dim, int taps, float eps, int single) {
+    __shared__ float inv[RUN + CONV_TAPS];
+    __shared__ float scratch[33];
+    pdl_wait();
+    pdl_trigger();
+    const int r0 = blockIdx.x * RUN, r1 = min(rows, r0 + RUN), lo = single ? r0 : max(0, r0 - (taps - 1));
+    if constexpr (RUN == 1) {
+        // (one row: all of the block's threads on it; in a step with portions RUN is larger)
+        float ss = 0.f;
+        for (int i = threadIdx.x * V; i < dim; i += blockDim.x * V) {
+            const Pack<V> v = load_pack<V>(x + (size_t)r0 * dim + i);
+#pragma unroll
+            for (int k = 0; k < V; ++k) ss = fmaf(v.v[k], v.v[k], ss);
+        }
+        ss = block_sum(ss, scratch);
+        if (threadIdx.x == 0) inv[0] = 1.f / sqrtf(ss / (float)dim + eps);
+    } else {
+        rms_factors(x, lo, r1, dim, eps, inv);
+    }
+    __syncthreads();
+    for (int i = threadIdx.x * V; i < dim; i += blockDim.x * V) {
+        float g[V];
+#pragma unroll
+        for (int k = 0; k < V; ++k) g[k] = gain[i + k];
+        auto normed = [&](int r) {
+            Pack<V> h = load_pack<V>(x + (size_t)r * dim + i);
+            const float f = inv[r - lo];
+#pragma unroll
+            for (int k = 0; k < V; ++k) h.v[k] = __fmul_rn(__fmul_rn(h.v[k], f), g[k]);
+            return h;
+        };
+        for (int r = r0; r < r1; ++r) {
+            const int seg = row_seg[r], slot = state_slots[seg], t = single ? 0 : r - seg_start[seg];
+            const bool ok = jllm_in_bounds(slot, num_slots, BOUNDS_SLOT);
+            float* st = state + (size_t)(ok ? slot : 0) * max(taps - 1, 1) * dim + i;
+            const Pack<V> h = normed(r);
+            Pack<V> acc = h;
+            for (int j = 0; j < taps; ++j) {
+                const int at = t - (taps - 1) + j;
+                Pack<V> in;
+                if (j == taps - 1) in = h;
+                else if (at >= 0) in = normed(r - (taps - 1) + j);
+                else if (ok) in = load_pack<V>(st + (size_t)(taps - 1 + at) * dim);
+                else {
+#pragma unroll
+                    for (int k = 0; k < V; ++k) in.v[k] = 0.f;
+                }
+#pragma unroll
+                for (int k = 0; k < V; ++k) acc.v[k] = fmaf(conv[(i + k) * taps + j], in.v[k], acc.v[k]);
+                // a step of single rows: this thread alone touches these channels of the slot; entry j - 1 has been read
+                if (single && j > 0 && ok) store_pack<V>(st + (size_t)(j - 1) * dim, in);
+            }
+            store_pack<V>(out + (size_t)r * dim + i, acc);
+        }
+    }
+}
+
+// behind it, for steps with portions: the state's new entry j is the normed row of local index n - (taps - 1) + j
+__global__ void __launch_bounds__(256)
+norm_conv_save_kernel(const float* __restrict__ x, VecRef gain, float* __restrict__ state, int num_slots,
+                      const int* __restrict__ seg_start, const int* __restrict__ seg_len, const int* __restrict__ state_slots,
+                      int dim, int taps, float eps) {
+    __shared__ float inv[CONV_TAPS];
+    pdl_wait();
+    pdl_trigger();
+    const int seg = blockIdx.x, first = seg_start[seg], n = seg_len[seg], slot = state_slots[seg];
+    if (n <= 0 || !jllm_in_bounds(slot, num_slots, BOUNDS_SLOT)) return;
+    float* st = state + (size_t)slot * (taps - 1) * dim;
+    const int lo = max(0, n - (taps - 1));
+    rms_factors(x, first + lo, first + n, dim, eps, inv);
+    __syncthreads();
+    for (int i = threadIdx.x; i < dim; i += blockDim.x)
+        for (int j = 0; j + 1 < taps; ++j) {        // (ascending: the old entry j + n is read before it is written)
+            const int at = n - (taps - 1) + j;
+            st[(size_t)j * dim + i] = at >= 0 ? __fmul_rn(__fmul_rn(x[(size_t)(first + at) * dim + i], inv[at - lo]), gain[i])
+                                              : st[(size_t)(taps - 1 + at) * dim + i];
+        }
+}
+
 }  // namespace
 
 JLLM_BOUNDS_READER(residual_paths)
@@ -369,4 +511,35 @@ JLLM_EXPORT int jllm_scale_values(float* x, float s, long long count, cudaStream
     const int blocks = (int)min((size_t)65535, ((size_t)count + 255) / 256);
     jllm_launch(scale_values_kernel, dim3(blocks), dim3(256), 0, stream, LAUNCH_DEPENDENT, x, s, (size_t)count);
     return jllm_check_launch("scale_values");
+}
+
+// x [rows, dim] float32; gain [dim] and conv [dim, taps] of types `gain_dtype` and `conv_dtype`; state [slots, max(taps - 1, 1), dim]
+// float32; out [rows, dim] of type `out_dtype`.
+JLLM_EXPORT int jllm_norm_conv(const float* x, const void* gain, int gain_dtype, const void* conv, int conv_dtype, float* state,
+                               int num_slots, const int* row_seg, const int* seg_start, const int* seg_len,
+                               const int* state_slots, void* out, int out_dtype, int rows, int segments, int dim, int taps,
+                               float eps, int single, cudaStream_t stream) {
+    JLLM_REQUIRE(rows >= 0 && dim > 0 && taps >= 1 && taps <= CONV_TAPS, "norm_conv: rows=%d dim=%d taps=%d (at most %d)", rows, dim,
+                 taps, CONV_TAPS);
+    if (rows == 0) return JLLM_OK;
+    const VecRef g{gain, gain_dtype}, c{conv, conv_dtype};
+    const bool vec = dim % 4 == 0 && (((uintptr_t)x | (uintptr_t)state | (uintptr_t)out) % 16) == 0;
+#define JLLM_NORM_CONV(T, RUN, V)                                                                                              \
+    jllm_launch(norm_conv_kernel<T, RUN, V>, dim3((rows + RUN - 1) / RUN), dim3(256), 0, stream, LAUNCH_DEPENDENT, x, g, c, state,  \
+                num_slots, row_seg, seg_start, state_slots, (T*)out, rows, dim, taps, eps, single)
+#define JLLM_NORM_CONV_T(T)                                                                                                    \
+    do {                                                                                                                       \
+        if (single && vec) JLLM_NORM_CONV(T, 1, 4);                                                                            \
+        else if (single) JLLM_NORM_CONV(T, 1, 1);                                                                              \
+        else if (vec) JLLM_NORM_CONV(T, CONV_RUN, 4);                                                                          \
+        else JLLM_NORM_CONV(T, CONV_RUN, 1);                                                                                   \
+    } while (0)
+    if (out_dtype == JLLM_F32) JLLM_NORM_CONV_T(float);
+    else JLLM_NORM_CONV_T(__nv_bfloat16);
+#undef JLLM_NORM_CONV_T
+#undef JLLM_NORM_CONV
+    if (!single && taps > 1)
+        jllm_launch(norm_conv_save_kernel, dim3(segments), dim3(256), 0, stream, LAUNCH_DEPENDENT, x, g, state, num_slots, seg_start,
+                    seg_len, state_slots, dim, taps, eps);
+    return jllm_check_launch("norm_conv");
 }

@@ -10,11 +10,12 @@ left unread, as the reference's converter drops it: model/ModelConverter.java:66
 """
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import Dict, List, Optional
 
 import torch
 
-from ..cache.manager import needs_of
+from ..cache.manager import PagedKeysValues, needs_of, span_covering
 from ..config.specs import ConfigError, Decoder
 from ..csrc import ops
 from ..parts import Linear, RunCache, Runtime, part_class
@@ -109,6 +110,17 @@ class DecoderModel:
             need = None if run.cache_of is not None else part_class("mixer", mixer.kind).cache_need(mixer)
             own = needs_of(self._block_need(self.spec, layer))       # the arrangement's own: kept by every run, borrower or not
             needs.append(tuple(needs_of(need)) + tuple(own) if own else need)
+        # a run that reads another run's rows under a mask of its own: the owner keeps what either of them may still see
+        for run in self.spec.schedule:
+            if run.cache_of is None:
+                continue
+            mixer = self.spec.layers[run.layer].mixer
+            theirs = [n for n in needs_of(part_class("mixer", mixer.kind).cache_need(mixer)) if isinstance(n, PagedKeysValues)]
+            held = needs_of(needs[run.cache_of])
+            kept = tuple(replace(n, window=span_covering(n.window, theirs[0].window), keep_first=max(n.keep_first, theirs[0].keep_first) if n.window > 0 else 0)
+                         if theirs and isinstance(n, PagedKeysValues) else n for n in held)
+            if kept != held:
+                needs[run.cache_of] = kept
         return needs
 
     def _run_cache(self, cache, i: int) -> RunCache:

@@ -9,6 +9,7 @@ from .mlp import DenseGlu, DenseMlp
 from .linear_attention import FixedDecayLinearAttention, GatedLinearAttention
 from .state_space import SelectiveStateSpace
 from .matrix_memory import MatrixMemory
+from .delta_rule import GeneralDelta
 from .parallel import ParallelMixers
 from .latent_attention import LatentAttention
 from .experts import RoutedExperts

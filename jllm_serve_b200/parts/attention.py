@@ -20,6 +20,15 @@ positions; the cache never gives their pages back); a learned sink per query hea
 softmax's denominator without a key or a value; a sigmoid gate of FULL width (one gate value per value of the concatenated
 heads, `gate = "sigmoid"`), whose rows also ride at the end of the stacked projection; and `out_scale`, a factor on the
 mixer's result that a mixer of mixers sets (applied together with the gate, in front of the output projection).
+
+And the WIDE forms (`spec.wide`), whose rows another kernel prepares (`ops.map_prepare`): an RMS norm over all query (key) columns
+of a row at once; a stored factor per query head on the scores (folded into the query gains, which multiply the same values, when
+the part is built); and a differential attention of two maps per head over the same values. The two maps cost one pass and one
+copy of the values: a cached key row holds [map 1, map 2], a query head becomes two rows [q1, 0] and [0, q2] of that width, so the
+attention kernels see heads x 2 query heads over kv_heads plain heads; `ops.map_difference` then subtracts the second map's
+result (times lambda, a number of the layer made from four stored vectors), norms the difference per head and scales it. Rows are
+filled up with zeros to a width the tile kernels take where that costs little (`spec.row_dim`). With `own_kv` False there are no
+key and value projections: the run reads what another run cached, under its own mask.
 """
 from __future__ import annotations
 
@@ -43,6 +52,15 @@ class GqaAttention(Mixer):
     def __init__(self, spec, dim: int, tensors: dict, prefix: str, runtime, rope=None):
         self.spec, self.dim, self.rt, self.rope = spec, dim, runtime, rope
         self.overwrite, self.out_scale = False, 1.0
+        # what the attention kernels are told about the keys a row sees: 0 all, w > 0 a window, -c < 0 chunks of c positions
+        self.span = -spec.chunk if spec.chunk else spec.window
+        self.keep_first = int(getattr(spec, "keep_first", 0))
+        self.wide = spec.wide
+        if rope is not None and rope.rotary_dim > spec.head_dim:
+            raise ValueError(f"rotary_dim={rope.rotary_dim} exceeds head_dim={spec.head_dim}")
+        if self.wide:
+            self._build_wide(tensors, prefix)
+            return
         H, Hkv, hd, vd, names = spec.heads, spec.kv_heads, spec.head_dim, spec.v_dim, spec.names
         self.q_width, self.k_width, self.v_width = H * hd, Hkv * hd, Hkv * vd
         self.gated = spec.gate in ("head_sigmoid", "sigmoid")
@@ -79,16 +97,70 @@ class GqaAttention(Mixer):
         del w, b
         self.out = Linear(tensors.pop(prefix + names.o), tensors.pop(prefix + names.o_bias) if spec.out_bias else None)
         self.sink = tensors.pop(prefix + names.sink) if spec.sink else None
-        self.keep_first = int(getattr(spec, "keep_first", 0))
         self.q_gain = tensors.pop(prefix + names.q_norm) if spec.qk_norm else None
         self.k_gain = tensors.pop(prefix + names.k_norm) if spec.qk_norm else None
-        if rope is not None and rope.rotary_dim > hd:
-            raise ValueError(f"rotary_dim={rope.rotary_dim} exceeds head_dim={hd}")
-        # what the attention kernels are told about the keys a row sees: 0 all, w > 0 a window, -c < 0 chunks of c positions
-        self.span = -spec.chunk if spec.chunk else spec.window
+
+    def _build_wide(self, tensors: dict, prefix: str) -> None:
+        s, names = self.spec, self.spec.names
+        q_width, k_width, v_width = s.heads * s.maps * s.head_dim, s.kv_heads * s.maps * s.head_dim, s.kv_heads * s.v_dim
+        w = [tensors.pop(prefix + names.q)]
+        self.k_off, self.v_off, self.width = 0, 0, q_width
+        if s.own_kv:
+            rows, at = [], 0
+            for t, n in ((w[0], q_width), (tensors.pop(prefix + names.k), k_width), (tensors.pop(prefix + names.v), v_width)):
+                if at != _up8(at):       # every piece starts at a multiple of 8 columns
+                    rows.append(torch.zeros((_up8(at) - at, self.dim), dtype=t.dtype, device=t.device))
+                    at = _up8(at)
+                rows.append(t)
+                self.k_off, self.v_off = self.v_off, at
+                at += n
+            w, self.width = rows, at
+        self.qkv = Linear(torch.cat(w, dim=0).contiguous())
+        del w
+        W, vd = s.row_dim, s.v_dim
+        out = tensors.pop(prefix + names.o)
+        if s.maps == 1 and W != vd:
+            # the attention's result keeps the rows' width; its tail (zeros) meets columns of zeros
+            wide = torch.zeros((self.dim, s.heads, W), dtype=out.dtype, device=out.device)
+            wide[:, :, :vd] = out.view(self.dim, s.heads, vd)
+            out = wide.view(self.dim, s.heads * W).contiguous()
+        self.out = Linear(out)
+        self.q_gain = self.k_gain = None
+        if s.qk_norm:
+            self.q_gain = tensors.pop(prefix + names.q_norm).float()
+            self.k_gain = tensors.pop(prefix + names.k_norm).float().contiguous() if s.own_kv else None
+        if s.head_scale:
+            factor = tensors.pop(prefix + names.head_scale).float().repeat_interleave(s.maps * s.head_dim)
+            if self.q_gain is None:
+                raise ValueError("a factor per head on the scores is built together with a norm over all heads")
+            self.q_gain = self.q_gain * factor
+        self.q_gain = self.q_gain.contiguous() if self.q_gain is not None else None
+        self.lam = 0.0
+        if s.maps == 2:
+            q1, k1, q2, k2 = (tensors.pop(prefix + n).double() for n in names.lambdas)
+            self.lam = float((torch.exp((q1 * k1).sum()) - torch.exp((q2 * k2).sum())).item()) + s.diff
+
+    @classmethod
+    def _wide_wants(cls, s, dim: int, prefix: str) -> dict:
+        names = s.names
+        q_width, k_width = s.heads * s.maps * s.head_dim, s.kv_heads * s.maps * s.head_dim
+        out = {prefix + names.q: TensorWant((q_width, dim)), prefix + names.o: TensorWant((dim, s.heads * s.v_dim))}
+        if s.own_kv:
+            out.update({prefix + names.k: TensorWant((k_width, dim)), prefix + names.v: TensorWant((s.kv_heads * s.v_dim, dim))})
+        if s.qk_norm:
+            out[prefix + names.q_norm] = TensorWant((q_width,), "vector", init="gain")
+            if s.own_kv:
+                out[prefix + names.k_norm] = TensorWant((k_width,), "vector", init="gain")
+        if s.head_scale:
+            out[prefix + names.head_scale] = TensorWant((s.heads,), "vector", init="gain")
+        if s.maps == 2:
+            out.update({prefix + n: TensorWant((s.head_dim,), "vector") for n in names.lambdas})
+        return out
 
     @classmethod
     def wants(cls, spec, dim: int, prefix: str) -> dict:
+        if spec.wide:
+            return cls._wide_wants(spec, dim, prefix)
         H, Hkv, hd, vd, names = spec.heads, spec.kv_heads, spec.head_dim, spec.v_dim, spec.names
         out = {prefix + names.q: TensorWant((H * hd, dim)),
                prefix + names.k: TensorWant((Hkv * hd, dim)),
@@ -115,11 +187,13 @@ class GqaAttention(Mixer):
     def cache_need(cls, spec):
         # a cache row holds a key in its first head_dim values and a value in its first value_dim; under a chunk mask the
         # pages of chunks that have passed are given back as under a window (the need's window is then -chunk)
-        return PagedKeysValues(spec.kv_heads, max(spec.head_dim, spec.v_dim), -spec.chunk if spec.chunk else spec.window,
+        return PagedKeysValues(spec.kv_heads, spec.row_dim, -spec.chunk if spec.chunk else spec.window,
                                keep_first=int(getattr(spec, "keep_first", 0)))
 
     def _tiles_fit(self) -> bool:
         s = self.spec
+        if self.wide:
+            return ops.attention_decode_fits(self.rt.dtype, s.heads * s.maps, s.kv_heads, s.row_dim)
         return (s.v_dim == s.head_dim and ops.attention_decode_fits(self.rt.dtype, s.heads, s.kv_heads, s.head_dim)
                 and ops.attention_tiles_take(self.keep_first, self.sink))
 
@@ -128,9 +202,34 @@ class GqaAttention(Mixer):
         if not self._tiles_fit():
             return 1                   # the plain attention's launches do not depend on the context
         scratch = self.rt.buffer("attention_scratch", 2 << 20, torch.float32, rows=1)[0]
-        return ops.decode_bucket_cap(rows, s.kv_heads, s.heads, s.head_dim, self.span, scratch)
+        heads, width = (s.heads * s.maps, s.row_dim) if self.wide else (s.heads, s.head_dim)
+        return ops.decode_bucket_cap(rows, s.kv_heads, heads, width, self.span, scratch)
+
+    def _forward_wide(self, xb, x, batch, cache) -> None:
+        s, rows, rope, W = self.spec, xb.shape[0], self.rope, self.spec.row_dim
+        if cache.writes != s.own_kv:
+            raise ops.KernelError("an attention without key and value projections reads another run's cache, one with them its own")
+        qkv = self.rt.buffer("qkv", self.width)[:rows]
+        self.qkv.forward(xb, qkv)
+        heads = s.heads * s.maps
+        q = self.rt.buffer("map_queries", heads * W)[:rows]
+        ops.map_prepare(qkv, self.k_off, self.v_off, self.q_gain, self.k_gain, s.qk_norm_eps, rope.cos if rope else None,
+                        rope.sin if rope else None, rope.rotary_dim if rope else 0, rope.pairing if rope else "half",
+                        batch.positions, batch.slots[cache.group] if cache.writes else None, q, cache.keys, cache.values, s.heads,
+                        s.kv_heads, s.maps, s.head_dim, s.v_dim, W, self.rt.page_size, write_kv=cache.writes)
+        att = self.rt.buffer("attention_out", heads * W)[:rows]
+        scratch = self.rt.buffer("attention_scratch", 2 << 20, torch.float32, rows=1)[0]
+        ops.attention(q, cache.keys, cache.values, att, batch, cache.group, heads, s.kv_heads, W, self.rt.page_size, self.span,
+                      s.scale, scratch, keep_first=self.keep_first)
+        if s.maps == 2:
+            y = self.rt.buffer("map_difference", s.heads * s.v_dim)[:rows]
+            ops.map_difference(att, W, self.lam, s.diff_norm_eps, 1.0 - s.diff, y, s.heads, s.v_dim)
+            att = y
+        self.out.forward(att, x, accumulate=not self.overwrite)
 
     def forward(self, xb, x, batch, cache) -> None:
+        if self.wide:
+            return self._forward_wide(xb, x, batch, cache)
         s, rows = self.spec, xb.shape[0]
         if cache.writes or not self.classic or self.gated:
             qkv = self.rt.buffer("qkv", self.width)[:rows]

@@ -8,7 +8,10 @@ is the epilogue of their last matrix product).
 Two things a layer spec may say beyond that: `feed_forward=None` (the layer is its mixer alone, and has no second
 norm), and `residual_scale` s (x += s * part(norm(x))). A part that can scale its own result says so
 (`takes_residual_scale`; it gets the factor as `residual_scale` and applies it in front of its last product); any other
-part adds into a zeroed float32 buffer instead, which is then added to x with the factor.
+part adds into a zeroed float32 buffer instead, which is then added to x with the factor. And `input_conv` (`pre_norm` only):
+what the mixer reads is its normed rows plus a short causal convolution over them, h_t + sum_j c[:, j] h_(t - taps + 1 + j); the
+norm and the convolution are one launch (`ops.norm_conv`), and the block keeps a request's last taps - 1 normed rows between
+steps (`cache_need`: a state of its own beside the mixer's, float32, zero for a new request).
 """
 from __future__ import annotations
 
@@ -21,6 +24,8 @@ from .base import Block, part_class, register_block
 
 
 class PreNormBlock(Block):
+    takes_input_conv = True
+
     def __init__(self, spec, dim: int, tensors: dict, prefix: str, runtime, position_encodings):
         names = spec.names
         norm_cls = part_class("norm", spec.norm.kind)
@@ -37,6 +42,11 @@ class PreNormBlock(Block):
             self.ffn_norm = norm_cls(spec.norm, dim, tensors, prefix + names.feed_forward_norm, runtime)
             self.feed_forward = part_class("feed_forward", spec.feed_forward.kind)(
                 spec.feed_forward, dim, tensors, prefix + names.feed_forward, runtime)
+        self.input_conv = None
+        if spec.input_conv:
+            if not type(self).takes_input_conv or spec.norm.kind != "rmsnorm":
+                raise ValueError("a convolution over the mixer's input is built for the pre_norm arrangement with an RMS norm")
+            self.input_conv = tensors[prefix + spec.input_conv]
         self.scale = float(getattr(spec, "residual_scale", 1.0))
         self._scaled_outside = set()
         for part in (self.mixer, self.feed_forward):
@@ -57,10 +67,17 @@ class PreNormBlock(Block):
         return getattr(self.mixer, "decode_bucket_cap", lambda _: 32)(rows)
 
     @classmethod
+    def cache_need(cls, spec, dim: int):
+        """What the arrangement itself keeps between steps, beside its mixer's need."""
+        return FixedState((max(spec.input_conv_taps - 1, 1), dim), "float32") if spec.input_conv else None
+
+    @classmethod
     def wants(cls, spec, dim: int, prefix: str) -> dict:
         names = spec.names
         norm_cls = part_class("norm", spec.norm.kind)
         out = {}
+        if spec.input_conv:
+            out[prefix + spec.input_conv] = TensorWant((dim, spec.input_conv_taps), "vector")
         out.update(norm_cls.wants(spec.norm, dim, prefix + names.mixer_norm))
         out.update(part_class("mixer", spec.mixer.kind).wants(spec.mixer, dim, prefix + names.mixer))
         if spec.feed_forward is not None:
@@ -83,7 +100,10 @@ class PreNormBlock(Block):
 
     def forward(self, x, batch, cache) -> None:
         xb = self.rt.buffer("normed", self.dim)[:x.shape[0]]
-        self.mixer_norm.forward(x, xb)
+        if self.input_conv is not None:
+            ops.norm_conv(x, self.mixer_norm.gain, self.mixer_norm.eps, self.input_conv, cache.block_states[0], batch, xb)
+        else:
+            self.mixer_norm.forward(x, xb)
         y = self._into(self.mixer, x)
         self.mixer.forward(xb, y, batch, cache)
         self._settle(x, y)
@@ -105,6 +125,7 @@ class ParallelResidualBlock(PreNormBlock):
 
     Both parts add into the float32 stream themselves, one after the other (the add is the epilogue of their last products);
     neither reads what the other wrote, because both read h. The layer's one gain is `names.mixer_norm`."""
+    takes_input_conv = False
 
     def __init__(self, spec, dim: int, tensors: dict, prefix: str, runtime, position_encodings):
         if spec.feed_forward is not None and spec.names.feed_forward_norm != spec.names.mixer_norm:
@@ -138,6 +159,7 @@ class SandwichNormBlock(PreNormBlock):
     the buffer zeroed), and one kernel norms it, adds it to the stream and also makes the normed input of the part that
     follows: the feed-forward's, or the next block's mixer's (`ops.norm_chain`; the model hands a block the next block's
     gain where both arrange their norms this way)."""
+    takes_input_conv = False
 
     def __init__(self, spec, dim: int, tensors: dict, prefix: str, runtime, position_encodings):
         super().__init__(spec, dim, tensors, prefix, runtime, position_encodings)

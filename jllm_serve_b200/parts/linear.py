@@ -39,11 +39,17 @@ class Linear:
             out.packed = ops.pack_weight(self.packed.unpack()[lo:hi].contiguous())
         return out
 
-    def forward(self, a: torch.Tensor, out: torch.Tensor, accumulate: bool = False, swiglu: bool = False) -> None:
+    def forward(self, a: torch.Tensor, out: torch.Tensor, accumulate: bool = False, swiglu: bool = False,
+                relu2: bool = False) -> None:
         """a [rows, in] (compute dtype) -> out [rows, out]; `accumulate` adds into out (the float32 residual);
+        `relu2` stores max(result, 0)^2 (behind the bias) instead of the result;
         `swiglu`: the weight's rows are interleaved gate / up blocks and out is [rows, out / 2]."""
         if a.shape[0] == 0:
             return
+        if relu2:
+            if accumulate or swiglu:
+                raise ops.KernelError("relu squared in a product's epilogue goes with a stored result only")
+            accumulate = ops.EPILOGUE_RELU2
         if self.packed is not None and ops.gemm_bf16_fits(a, self.packed, out):
             ops.gemm_bf16(a, self.packed, out, self.bias, accumulate, swiglu)
         elif swiglu:
