@@ -13,7 +13,7 @@ read (every weight once plus the cache of the live requests) with the measured c
 `points` holds decode at batch 1 and 64; `check` compares the bfloat16 logits with the 32-bit path's at these
 layer sizes (two layers, untimed). Peaks come from MEASURED_PEAKS.json when it exists.
 
-`--design madevik`, `--design movivik`, `--design bozevik` and `--design guvolix` are another program under the same roof and leave the default
+`--design madevik`, `--design movivik`, `--design bozevik`, `--design guvolix` and `--design fusazen` are another program under the same roof and leave the default
 workload alone: prefill and decode of the Madevik design (gated linear attention, attention over a cached latent, routed
 experts), of the Movivik design (chunked and parallel attention layers, linear attention with fixed decays, norms in front of
 and behind every part) or of the Bozevik design (attention over a cached latent with a query latent and a shared rotated key
@@ -197,6 +197,25 @@ def guvolix_shape(width, heads, kv_heads, ff, runs, window=1024, keep=64, vocab=
             "layers": layers}
 
 
+def fusazen_shape(width, heads, kv_heads, ff, runs, chunk=1024, vocab=32768):
+    """Layers in fours: an attention whose queries and keys are normed over all heads (heads of 128), a delta rule (heads of 64 key
+    and value channels, a decay projection of rank 64), a differential attention (two maps of 64 values per head over values of
+    128, half of each map rotated) and one that reads its keys and values; chunk masks of `chunk` positions; relu-squared
+    feed-forwards with biases of `ff` hidden values."""
+    mlp = {"kind": "dense", "ff": ff}
+    att2 = {"type": "attention_2", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128,
+                                                         "scale": 128 ** -0.5, "mask": {"size": chunk}}}
+    delta = {"type": "general_delta", "mlp": mlp, "mixer": {"heads": width // 64, "dim": 64, "decay_rank": 64}}
+    diff = {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "mask": {"size": chunk}, "diff": 0.5,
+            "rot": {"base": 10000.0, "dims": 32}}
+    layers = []
+    for i in range(runs):
+        layers.append([att2, delta, {"type": "attention", "mlp": mlp, "mixer": diff},
+                       {"type": "attention", "mlp": mlp, "mixer": dict(diff, kv_from=i - 1)}][i % 4])
+    return {"architecture": "Fusazen", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "canon": {"taps": 4},
+            "embedding": {"scale": 2.0}, "layers": layers}
+
+
 def movivik_parallel_shape(width, heads, kv_heads, ff, runs, vocab=32768):
     """A Movivik model of parallel layers only (the closest kin of the Guvolix shape): a causal attention beside linear
     attention with a fixed decay per head, heads of 128, a dense gated feed-forward."""
@@ -228,6 +247,12 @@ DESIGN_SIZES = {
                           movivik_parallel_shape(2048, 16, 8, 8192, 8), "movivik_parallel"),
                 "w4096": (guvolix_shape(4096, 32, 8, 12288, 4), _qwen3_shape(4096, 4, 32, 8, 12288),
                           movivik_parallel_shape(4096, 32, 8, 12288, 4), "movivik_parallel")},
+    # feed-forwards of 1.5 times the gated ones' hidden values (two matrices instead of three); beside each the Qwen3 shape and
+    # a Movivik model (chunked attention layers, and layers of attention beside linear attention)
+    "fusazen": {"w2048": (fusazen_shape(2048, 16, 8, 12288, 8), _qwen3_shape(2048, 8, 16, 8, 8192),
+                          movivik_shape(2048, 16, 8, 8192, 8), "movivik"),
+                "w4096": (fusazen_shape(4096, 32, 8, 18432, 4), _qwen3_shape(4096, 4, 32, 8, 12288),
+                          movivik_shape(4096, 32, 8, 12288, 4), "movivik")},
 }
 
 
@@ -333,10 +358,10 @@ def _tensors_of(obj, seen=None):
 
 def main() -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawTextHelpFormatter)
-    ap.add_argument("--design", default="", choices=["", "madevik", "movivik", "bozevik", "guvolix"],
-                    help="madevik, movivik, bozevik, guvolix: time that design beside the Qwen3 dense shape of equal size (bozevik: "
+    ap.add_argument("--design", default="", choices=["", "madevik", "movivik", "bozevik", "guvolix", "fusazen"],
+                    help="madevik, movivik, bozevik, guvolix, fusazen: time that design beside the Qwen3 dense shape of equal size (bozevik: "
                          "also beside a Madevik model of latent-attention layers; guvolix: also beside a Movivik model of "
-                         "parallel layers) instead of the default workload")
+                         "parallel layers; fusazen: also beside a Movivik model) instead of the default workload")
     ap.add_argument("--design-sizes", default="w2048,w4096", help="which of the sizes of --design, with commas between them")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=64)

@@ -51,12 +51,38 @@ struct DeltaSource {
     int ld, r_off, k_off, v_off, a_off;
 };
 
+// The norm and gate behind the recurrence, y[r, h] = o[r, h] / sqrt(mean(o[r, h]^2) + eps) * gain * sigmoid(gate): taken along where
+// a block holds all of a head's value columns (y null: the results leave as they are, in `o`).
+struct DeltaNorm {
+    const float* gate;       // [rows, ld]
+    void* y;                 // [rows, heads * dv] of type `dtype`, or null
+    VecRef gain;             // [heads * dv]
+    float eps;
+    int ld, dtype;
+};
+
+// one warp: the dv results of (row, head) in shared memory -> y
+__device__ __forceinline__ void head_norm_row(const DeltaNorm& nm, const float* res, size_t row, int h, int heads, int dv) {
+    const int lane = threadIdx.x & 31;
+    float ss = 0.f;
+    for (int i = lane; i < dv; i += 32) ss = fmaf(res[i], res[i], ss);
+    ss = warp_sum(ss);
+    const float inv = 1.f / sqrtf(ss / (float)dv + nm.eps);
+    const float* g = nm.gate + row * nm.ld + (size_t)h * dv;
+    const size_t at = row * ((size_t)heads * dv) + (size_t)h * dv;
+    for (int i = lane; i < dv; i += 32) {
+        const float v = __fmul_rn(__fmul_rn(__fmul_rn(res[i], inv), nm.gain[h * dv + i]), sigmoid_f(g[i]));
+        if (nm.dtype == JLLM_F32) static_cast<float*>(nm.y)[at + i] = v;
+        else static_cast<__nv_bfloat16*>(nm.y)[at + i] = __float2bfloat16_rn(v);
+    }
+}
+
 // ---- token by token -----------------------------------------------------------------------------------------------------
 template <int LS, int R, int CB, int TOK>
 __global__ void __launch_bounds__(LS * CB)
 delta_recurrent_kernel(DeltaSource src, float* __restrict__ state, int num_slots, const int* __restrict__ seg_start,
-                       const int* __restrict__ seg_len, const int* __restrict__ state_slots, float* __restrict__ o, int heads,
-                       int dk, int dv) {
+                       const int* __restrict__ seg_len, const int* __restrict__ state_slots, float* __restrict__ o, DeltaNorm nm,
+                       int heads, int dk, int dv) {
     constexpr int DKP = LS * R, THREADS = LS * CB;
     extern __shared__ __align__(16) float smem[];
     float* ks = smem;                    // [TOK][DKP] k
@@ -65,12 +91,14 @@ delta_recurrent_kernel(DeltaSource src, float* __restrict__ state, int num_slots
     float* as = rs + TOK * DKP;          //            a k
     float* vs = as + TOK * DKP;          // [TOK][CB]
     float* inv2 = vs + TOK * CB;         // [TOK]      1 / (sum(k^2) + 1e-6)
-    pdl_wait();
-    pdl_trigger();
+    float* res = inv2 + TOK;             // [TOK][CB]  results on their way to the norm
     const int seg = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * CB;
     const int tid = threadIdx.x, l = tid % LS, c = tid / LS, j = c0 + c;
     const int first = seg_start[seg], n = seg_len[seg], slot = state_slots[seg];
-    if (!jllm_in_bounds(slot, num_slots, BOUNDS_SLOT)) return;
+    if (!jllm_in_bounds(slot, num_slots, BOUNDS_SLOT)) {
+        pdl_wait();
+        return;
+    }
     float* S = state + (((size_t)slot * heads + h) * dk) * dv;
     float s[R];
 #pragma unroll
@@ -78,6 +106,10 @@ delta_recurrent_kernel(DeltaSource src, float* __restrict__ state, int num_slots
         const int i = 4 * (l + LS * (r >> 2)) + (r & 3);
         s[r] = (i < dk && j < dv) ? S[(size_t)i * dv + j] : 0.f;
     }
+    // The step's tables and a slot's state are older than the kernel in front of this one (nothing between a slot's opening or
+    // its last step and this launch is so close), so the state is on its way before that kernel's results are waited for.
+    pdl_wait();
+    pdl_trigger();
     for (int t0 = 0; t0 < n; t0 += TOK) {
         const int nt = min(TOK, n - t0);
         for (int e = tid; e < nt * DKP; e += THREADS) {
@@ -142,9 +174,14 @@ delta_recurrent_kernel(DeltaSource src, float* __restrict__ state, int num_slots
             float acc = acc0 + acc1;
 #pragma unroll
             for (int m = 1; m < LS; m <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, m);
-            if (l == 0 && j < dv) o[(size_t)(first + t0 + t) * ((size_t)heads * dv) + (size_t)h * dv + j] = acc;
+            if (l == 0 && j < dv) {
+                if (nm.y != nullptr) res[t * CB + c] = acc;
+                else o[(size_t)(first + t0 + t) * ((size_t)heads * dv) + (size_t)h * dv + j] = acc;
+            }
         }
         __syncthreads();
+        if (nm.y != nullptr)         // (`res` is written again behind two more barriers)
+            for (int t = tid >> 5; t < nt; t += THREADS / 32) head_norm_row(nm, res + t * CB, (size_t)(first + t0 + t), h, heads, dv);
     }
 #pragma unroll
     for (int r = 0; r < R; ++r) {
@@ -155,14 +192,15 @@ delta_recurrent_kernel(DeltaSource src, float* __restrict__ state, int num_slots
 
 template <int LS, int R, int CB, int TOK>
 int launch_recurrent(const DeltaSource& src, float* state, int num_slots, const int* seg_start, const int* seg_len,
-                     const int* state_slots, float* o, int segments, int heads, int dk, int dv, cudaStream_t stream) {
-    const size_t smem = (size_t)(TOK * (4 * LS * R + CB) + TOK) * sizeof(float);
+                     const int* state_slots, float* o, const DeltaNorm& nm, int segments, int heads, int dk, int dv,
+                     cudaStream_t stream) {
+    const size_t smem = (size_t)(TOK * (4 * LS * R + 2 * CB) + TOK) * sizeof(float);
     auto kernel = delta_recurrent_kernel<LS, R, CB, TOK>;
     if (smem > 48 * 1024 &&
         cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
         return jllm_fail(JLLM_CUDA_ERROR, "delta_recurrent: %zu bytes of shared memory refused", smem);
     jllm_launch(kernel, dim3(segments, heads, (dv + CB - 1) / CB), dim3(LS * CB), smem, stream, LAUNCH_DEPENDENT, src, state,
-                num_slots, seg_start, seg_len, state_slots, o, heads, dk, dv);
+                num_slots, seg_start, seg_len, state_slots, o, nm, heads, dk, dv);
     return jllm_check_launch("delta_recurrent");
 }
 
@@ -203,10 +241,14 @@ __device__ __forceinline__ void tile_rows(float (&acc)[4][4], const float* A, co
     }
 }
 
-__global__ void __launch_bounds__(128)
+// D: the key and value width where both are that, known to the compiler; 0: read from the arguments
+constexpr int PREP_THREADS = 256;
+template <int D>
+__global__ void __launch_bounds__(PREP_THREADS, D == 64 ? 3 : 1)
 delta_chunk_prepare_kernel(DeltaSource src, const int* __restrict__ seg_start, const int* __restrict__ seg_len,
                            float* __restrict__ qp, float* __restrict__ o, float* __restrict__ M, float* __restrict__ N, int heads,
-                           int dk, int dv) {
+                           int dk_arg, int dv_arg) {
+    const int dk = D ? D : dk_arg, dv = D ? D : dv_arg;
     extern __shared__ __align__(16) float smem[];
     const int ldk = dk + 4, ldv = dv + 4;
     float* Bm = smem;                    // [C][ldk]  u_t e^(L_(t-1)), then W
@@ -222,7 +264,8 @@ delta_chunk_prepare_kernel(DeltaSource src, const int* __restrict__ seg_start, c
     pdl_trigger();
     const int seg = blockIdx.z, h = blockIdx.y, t0 = blockIdx.x * C, n = seg_len[seg];
     if (t0 >= n) return;
-    const int nt = min(C, n - t0), tid = threadIdx.x, threads = blockDim.x;
+    const int nt = min(C, n - t0), tid = threadIdx.x;
+    constexpr int threads = PREP_THREADS;
     const int first = seg_start[seg];
     const size_t row0 = (size_t)first + t0, hk = (size_t)heads * dk, hv = (size_t)heads * dv;
     const size_t chunk = (size_t)chunk_base(first, seg) + blockIdx.x;
@@ -306,74 +349,61 @@ delta_chunk_prepare_kernel(DeltaSource src, const int* __restrict__ seg_start, c
             }
     }
     __syncthreads();
-    // the triangular system, a thread per column: W from u_t e^(L_(t-1)), U from the values
+    // the triangular system (I + [u.au]) X = [u e^(L_(t-1)) | [u.k] V]: the values' right-hand side first, as a product ...
     const float *uau = sc, *uk = sc + C * LDS, *rau = sc + 2 * C * LDS, *rk = sc + 3 * C * LDS;
-    for (int col = tid; col < dk + dv; col += threads) {
-        float x[C];
-        const bool value = col >= dk;
-        float* mine = value ? Um + (col - dk) : Bm + col;
-        const int ldm = value ? ldv : ldk;
-        if (value) {
-            float v[C];
-#pragma unroll
-            for (int t = 0; t < C; ++t) v[t] = Vm[t * ldv + (col - dk)];
-#pragma unroll
-            for (int t = 0; t < C; ++t) {
-                float a0 = 0.f, a1 = 0.f;
-#pragma unroll
-                for (int s = 0; s < t; s += 4) {
-                    const float4 m = ld4(uau + t * LDS + s), w = ld4(uk + t * LDS + s);     // (zeros from s = t on)
-                    a0 = fmaf(w.x, v[s], a0);
-                    a1 = fmaf(-m.x, x[s], a1);
-                    if (s + 1 < t) { a0 = fmaf(w.y, v[s + 1], a0); a1 = fmaf(-m.y, x[s + 1], a1); }
-                    if (s + 2 < t) { a0 = fmaf(w.z, v[s + 2], a0); a1 = fmaf(-m.z, x[s + 2], a1); }
-                    if (s + 3 < t) { a0 = fmaf(w.w, v[s + 3], a0); a1 = fmaf(-m.w, x[s + 3], a1); }
-                }
-                x[t] = a0 + a1;
-            }
-        } else {
-#pragma unroll
-            for (int t = 0; t < C; ++t) {
-                float a0 = mine[t * ldm], a1 = 0.f;
-#pragma unroll
-                for (int s = 0; s < t; s += 4) {
-                    const float4 m = ld4(uau + t * LDS + s);
-                    a0 = fmaf(-m.x, x[s], a0);
-                    if (s + 1 < t) a1 = fmaf(-m.y, x[s + 1], a1);
-                    if (s + 2 < t) a0 = fmaf(-m.z, x[s + 2], a0);
-                    if (s + 3 < t) a1 = fmaf(-m.w, x[s + 3], a1);
-                }
-                x[t] = a0 + a1;
-            }
-        }
-#pragma unroll
-        for (int t = 0; t < C; ++t) mine[t * ldm] = x[t];
-    }
-    __syncthreads();
-    // what a token reads of the chunk's own tokens (O) and of the state in front of it (Q)
-    for (int tile = tid; tile < 8 * k4; tile += threads) {
-        const int ty = tile & 7, i0 = (tile >> 3) * 4;
-        float acc[4][4];
-#pragma unroll
-        for (int a = 0; a < 4; ++a) {
-            const float4 r = ld4(Rm + (ty + 8 * a) * ldk + i0);
-            acc[a][0] = r.x; acc[a][1] = r.y; acc[a][2] = r.z; acc[a][3] = r.w;
-        }
-        tile_rows<-1>(acc, rau, Bm, ldk, ty, i0);
-#pragma unroll
-        for (int a = 0; a < 4; ++a)
-            if (ty + 8 * a < nt)
-                st4(qp + (row0 + ty + 8 * a) * hk + (size_t)h * dk + i0, make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]));
-    }
     for (int tile = tid; tile < 8 * v4; tile += threads) {
         const int ty = tile & 7, i0 = (tile >> 3) * 4;
         float acc[4][4] = {};
-        tile_rows<1>(acc, rk, Vm, ldv, ty, i0);
-        tile_rows<-1>(acc, rau, Um, ldv, ty, i0);
+        tile_rows<1>(acc, uk, Vm, ldv, ty, i0);
+#pragma unroll
+        for (int a = 0; a < 4; ++a) st4(Um + (ty + 8 * a) * ldv + i0, make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]));
+    }
+    __syncthreads();
+    // ... then a thread per column, in place
+    for (int col = tid; col < dk + dv; col += threads) {
+        float* mine = col >= dk ? Um + (col - dk) : Bm + col;
+        const int ldm = col >= dk ? ldv : ldk;
+        float x[C];
+#pragma unroll
+        for (int t = 0; t < C; ++t) {
+            float a0 = mine[t * ldm], a1 = 0.f;
+#pragma unroll
+            for (int s = 0; s < t; s += 4) {
+                const float4 m = ld4(uau + t * LDS + s);         // (zeros from s = t on)
+                a0 = fmaf(-m.x, x[s], a0);
+                if (s + 1 < t) a1 = fmaf(-m.y, x[s + 1], a1);
+                if (s + 2 < t) a0 = fmaf(-m.z, x[s + 2], a0);
+                if (s + 3 < t) a1 = fmaf(-m.w, x[s + 3], a1);
+            }
+            x[t] = a0 + a1;
+            mine[t * ldm] = x[t];
+        }
+    }
+    __syncthreads();
+    // what a token reads of the state in front of the chunk (Q) and of the chunk's own tokens (O)
+    for (int tile = tid; tile < 8 * (k4 + v4); tile += threads) {
+        const bool own = tile >= 8 * k4;
+        const int ty = tile & 7, i0 = ((own ? tile - 8 * k4 : tile) >> 3) * 4;
+        float acc[4][4];
+        if (own) {
+#pragma unroll
+            for (int a = 0; a < 4; ++a) acc[a][0] = acc[a][1] = acc[a][2] = acc[a][3] = 0.f;
+            tile_rows<1>(acc, rk, Vm, ldv, ty, i0);
+            tile_rows<-1>(acc, rau, Um, ldv, ty, i0);
+        } else {
+#pragma unroll
+            for (int a = 0; a < 4; ++a) {
+                const float4 r = ld4(Rm + (ty + 8 * a) * ldk + i0);
+                acc[a][0] = r.x; acc[a][1] = r.y; acc[a][2] = r.z; acc[a][3] = r.w;
+            }
+            tile_rows<-1>(acc, rau, Bm, ldk, ty, i0);
+        }
 #pragma unroll
         for (int a = 0; a < 4; ++a)
-            if (ty + 8 * a < nt)
-                st4(o + (row0 + ty + 8 * a) * hv + (size_t)h * dv + i0, make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]));
+            if (ty + 8 * a < nt) {
+                float* dst = own ? o + (row0 + ty + 8 * a) * hv + (size_t)h * dv + i0 : qp + (row0 + ty + 8 * a) * hk + (size_t)h * dk + i0;
+                st4(dst, make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]));
+            }
     }
     // the chunk's transition M and what it adds, N
     float* Mc = M + (chunk * heads + h) * (size_t)dk * dk;
@@ -423,22 +453,28 @@ delta_chunk_prepare_kernel(DeltaSource src, const int* __restrict__ seg_start, c
 }
 
 // S <- M S + N through a portion's chunks, a block per (segment, head, 16 value columns); N of a chunk is replaced by the state
-// in front of it. M of the next chunk is on its way (cp.async, two buffers) while this one's product runs.
+// in front of it. M of the next chunks is on its way (cp.async, STAGES buffers) while this one's product runs.
+// A thread makes a 4 x 4 tile of the product over one of JS parts of the sum; the parts meet in shared memory.
 constexpr int WCB = 16;
-__global__ void __launch_bounds__(256)
+constexpr int WALK_THREADS = 256;
+template <int D, int STAGES, int JS>
+__global__ void __launch_bounds__(WALK_THREADS)
 delta_chunk_walk_kernel(const float* __restrict__ M, float* __restrict__ N, float* __restrict__ state, int num_slots,
                         const int* __restrict__ seg_start, const int* __restrict__ seg_len, const int* __restrict__ state_slots,
-                        int heads, int dk, int dv) {
+                        int heads, int dk_arg, int dv_arg) {
+    const int dk = D ? D : dk_arg, dv = D ? D : dv_arg;
     extern __shared__ __align__(16) float smem[];
     const int ldm = dk + 4, c0 = blockIdx.x * WCB, h = blockIdx.y, seg = blockIdx.z;
-    float* Ms = smem;                        // [2][dk][ldm]
-    float* Ns = Ms + 2 * dk * ldm;           // [2][dk][WCB]
-    float* Ss = Ns + 2 * dk * WCB;           // [dk][WCB]
+    float* Ms = smem;                        // [STAGES][dk][ldm]
+    float* Ns = Ms + STAGES * dk * ldm;      // [STAGES][dk][WCB]
+    float* Ss = Ns + STAGES * dk * WCB;      // [dk][WCB]
+    float* part = Ss + dk * WCB;             // [JS][dk][WCB]
     pdl_wait();
     pdl_trigger();
     const int first = seg_start[seg], n = seg_len[seg], slot = state_slots[seg];
     if (n <= 0 || !jllm_in_bounds(slot, num_slots, BOUNDS_SLOT)) return;
-    const int chunks = (n + C - 1) / C, tid = threadIdx.x, threads = blockDim.x, k4 = dk >> 2, cols = min(WCB, dv - c0);
+    constexpr int threads = WALK_THREADS;
+    const int chunks = (n + C - 1) / C, tid = threadIdx.x, k4 = dk >> 2, cols = min(WCB, dv - c0);
     const size_t base = (size_t)chunk_base(first, seg);
     float* S = state + (((size_t)slot * heads + h) * dk) * dv + c0;
     auto fetch = [&](int ch, int b) {
@@ -461,52 +497,65 @@ delta_chunk_walk_kernel(const float* __restrict__ M, float* __restrict__ N, floa
     for (int e = tid; e < dk * WCB; e += threads) {
         const int i = e / WCB, x = e - i * WCB;
         Ss[e] = x < cols ? S[(size_t)i * dv + x] : 0.f;
-        if (x >= cols) { Ns[e] = 0.f; Ns[dk * WCB + e] = 0.f; }
+        if (x >= cols)
+            for (int b = 0; b < STAGES; ++b) Ns[b * dk * WCB + e] = 0.f;
     }
-    fetch(0, 0);
-    const int ig = tid / (WCB / 2), cg = (tid % (WCB / 2)) * 2;
+#pragma unroll
+    for (int p = 0; p < STAGES - 1; ++p) {       // (an empty group where there is no such chunk: the counts stay the same)
+        if (p < chunks) fetch(p, p);
+        else asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    // this thread's tile: rows ig + k4 a, columns 4 cg .. 4 cg + 3; its part of the sum: groups of four [j_lo, j_hi)
+    const int tile = tid % (k4 * (WCB / 4)), jp = tid / (k4 * (WCB / 4)), ig = tile / (WCB / 4), cg = (tile % (WCB / 4)) * 4;
+    const int j_lo = jp * k4 / JS * 4, j_hi = (jp + 1) * k4 / JS * 4;
+    int b = 0;
     for (int ch = 0; ch < chunks; ++ch) {
-        const int b = ch & 1;
-        if (ch + 1 < chunks) {
-            fetch(ch + 1, b ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
+        // (the buffer that is filled now was read for the last time in front of the middle barrier of the turn before)
+        if (ch + STAGES - 1 < chunks) fetch(ch + STAGES - 1, b == 0 ? STAGES - 1 : b - 1);
+        else asm volatile("cp.async.commit_group;" ::: "memory");
+        asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 1) : "memory");
         __syncthreads();
         float* out = N + ((base + ch) * heads + h) * (size_t)dk * dv + c0;
         for (int e = tid; e < dk * (WCB / 4); e += threads) {
             const int i = e / (WCB / 4), x = (e - i * (WCB / 4)) * 4;
             if (x < cols) st4(out + (size_t)i * dv + x, ld4(Ss + i * WCB + x));
         }
-        float acc[4][2];
-        if (ig < k4) {
+        if (jp < JS) {
             const float* m = Ms + (size_t)b * dk * ldm;
+            float acc[4][4];
 #pragma unroll
             for (int a = 0; a < 4; ++a) {
-                const float2 v = *reinterpret_cast<const float2*>(Ns + b * dk * WCB + (ig + k4 * a) * WCB + cg);
-                acc[a][0] = v.x;
-                acc[a][1] = v.y;
+                const float4 v = jp == 0 ? ld4(Ns + b * dk * WCB + (ig + k4 * a) * WCB + cg) : make_float4(0.f, 0.f, 0.f, 0.f);
+                acc[a][0] = v.x; acc[a][1] = v.y; acc[a][2] = v.z; acc[a][3] = v.w;
             }
-#pragma unroll 4
-            for (int jx = 0; jx < dk; jx += 4) {
-                float2 sv[4];
-#pragma unroll
-                for (int q = 0; q < 4; ++q) sv[q] = *reinterpret_cast<const float2*>(Ss + (jx + q) * WCB + cg);
+#pragma unroll 2
+            for (int j = j_lo; j < j_hi; j += 4) {
+                const float4 s0 = ld4(Ss + j * WCB + cg), s1 = ld4(Ss + (j + 1) * WCB + cg), s2 = ld4(Ss + (j + 2) * WCB + cg),
+                             s3 = ld4(Ss + (j + 3) * WCB + cg);
 #pragma unroll
                 for (int a = 0; a < 4; ++a) {
-                    const float4 mv = ld4(m + (ig + k4 * a) * ldm + jx);
-                    acc[a][0] = fmaf(mv.w, sv[3].x, fmaf(mv.z, sv[2].x, fmaf(mv.y, sv[1].x, fmaf(mv.x, sv[0].x, acc[a][0]))));
-                    acc[a][1] = fmaf(mv.w, sv[3].y, fmaf(mv.z, sv[2].y, fmaf(mv.y, sv[1].y, fmaf(mv.x, sv[0].y, acc[a][1]))));
+                    const float4 mv = ld4(m + (ig + k4 * a) * ldm + j);
+                    fma4(acc[a], mv.x, s0);
+                    fma4(acc[a], mv.y, s1);
+                    fma4(acc[a], mv.z, s2);
+                    fma4(acc[a], mv.w, s3);
                 }
             }
-        }
-        __syncthreads();
-        if (ig < k4) {
 #pragma unroll
             for (int a = 0; a < 4; ++a)
-                *reinterpret_cast<float2*>(Ss + (ig + k4 * a) * WCB + cg) = make_float2(acc[a][0], acc[a][1]);
+                st4(part + (jp * dk + ig + k4 * a) * WCB + cg, make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]));
         }
+        __syncthreads();
+        for (int e = tid * 4; e < dk * WCB; e += threads * 4) {
+            float4 v = ld4(part + e);
+#pragma unroll
+            for (int p = 1; p < JS; ++p) {
+                const float4 w = ld4(part + p * dk * WCB + e);
+                v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+            }
+            st4(Ss + e, v);
+        }
+        b = b + 1 == STAGES ? 0 : b + 1;
     }
     __syncthreads();
     for (int e = tid; e < dk * WCB; e += threads) {
@@ -515,21 +564,37 @@ delta_chunk_walk_kernel(const float* __restrict__ M, float* __restrict__ N, floa
     }
 }
 
-// o_t += Q_t^T S0 for all chunks at once (N holds the states in front of the chunks)
+// o_t += Q_t^T S0 for all chunks at once (N holds the states in front of the chunks), and the norm and gate behind it (with
+// nm.y null the sums go back to o)
+template <int D>
 __global__ void __launch_bounds__(128)
 delta_chunk_out_kernel(const float* __restrict__ qp, const float* __restrict__ N, const int* __restrict__ seg_start,
-                       const int* __restrict__ seg_len, float* __restrict__ o, int heads, int dk, int dv) {
+                       const int* __restrict__ seg_len, float* __restrict__ o, DeltaNorm nm, int heads, int dk_arg, int dv_arg) {
+    const int dk = D ? D : dk_arg, dv = D ? D : dv_arg;
     extern __shared__ __align__(16) float smem[];
     const int ldk = dk + 4, ldv = dv + 4;
     float* Qs = smem;                    // [C][ldk]
     float* Ss = Qs + C * ldk;            // [dk][ldv]
+    float* Os = Ss + dk * ldv;           // [C][ldv]
     pdl_wait();
     pdl_trigger();
     const int seg = blockIdx.z, h = blockIdx.y, t0 = blockIdx.x * C, n = seg_len[seg];
     if (t0 >= n) return;
-    const int nt = min(C, n - t0), tid = threadIdx.x, threads = blockDim.x, k4 = dk >> 2, v4 = dv >> 2, first = seg_start[seg];
+    constexpr int threads = 128;
+    const int nt = min(C, n - t0), tid = threadIdx.x, k4 = dk >> 2, v4 = dv >> 2, first = seg_start[seg];
     const size_t row0 = (size_t)first + t0, hk = (size_t)heads * dk, hv = (size_t)heads * dv;
     const float* S = N + (((size_t)chunk_base(first, seg) + blockIdx.x) * heads + h) * (size_t)dk * dv;
+    // the norm's share of this thread: sixteen lanes a row, eight rows a turn; heads of 64 have their gates on the way from here on
+    const int sub = tid & 15, nrow = tid >> 4;
+    float4 gates[4];
+    if constexpr (D == 64) {
+        if (nm.y != nullptr) {
+#pragma unroll
+            for (int q = 0; q < 4; ++q)
+                gates[q] = nrow + 8 * q < nt ? ld4(nm.gate + (row0 + nrow + 8 * q) * nm.ld + (size_t)h * dv + sub * 4)
+                                             : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    }
     for (int e = tid; e < C * k4; e += threads) {
         const int t = e / k4, i = (e - t * k4) * 4;
         st4(Qs + t * ldk + i, t < nt ? ld4(qp + (row0 + t) * hk + (size_t)h * dk + i) : make_float4(0.f, 0.f, 0.f, 0.f));
@@ -561,11 +626,75 @@ delta_chunk_out_kernel(const float* __restrict__ qp, const float* __restrict__ N
         for (int a = 0; a < 4; ++a) {
             const int t = ty + 8 * a;
             if (t >= nt) continue;
-            float* dst = o + (row0 + t) * hv + (size_t)h * dv + j0;
-            const float4 old = ld4(dst);
-            st4(dst, make_float4(old.x + acc[a][0], old.y + acc[a][1], old.z + acc[a][2], old.w + acc[a][3]));
+            float* src = o + (row0 + t) * hv + (size_t)h * dv + j0;
+            const float4 old = ld4(src);
+            st4(nm.y != nullptr ? Os + t * ldv + j0 : src,
+                make_float4(old.x + acc[a][0], old.y + acc[a][1], old.z + acc[a][2], old.w + acc[a][3]));
         }
     }
+    if (nm.y == nullptr) return;
+    __syncthreads();
+    if constexpr (D == 64) {
+        float g[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) g[k] = nm.gain[h * dv + sub * 4 + k];
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+            const int t = nrow + 8 * q;
+            const float4 v = ld4(Os + t * ldv + sub * 4);        // (rows behind the portion's end: whatever lies there, not stored)
+            float ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+#pragma unroll
+            for (int m = 1; m < 16; m <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+            const float inv = 1.f / sqrtf(ss / (float)D + nm.eps);
+            const float r0 = v.x * inv * g[0] * sigmoid_f(gates[q].x), r1 = v.y * inv * g[1] * sigmoid_f(gates[q].y);
+            const float r2 = v.z * inv * g[2] * sigmoid_f(gates[q].z), r3 = v.w * inv * g[3] * sigmoid_f(gates[q].w);
+            if (t >= nt) continue;
+            const size_t at = (row0 + t) * hv + (size_t)h * dv + sub * 4;
+            if (nm.dtype == JLLM_F32) {
+                st4(static_cast<float*>(nm.y) + at, make_float4(r0, r1, r2, r3));
+            } else {
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(r0, r1), hi = __floats2bfloat162_rn(r2, r3);
+                uint2 u;
+                u.x = *reinterpret_cast<const uint32_t*>(&lo);
+                u.y = *reinterpret_cast<const uint32_t*>(&hi);
+                *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(nm.y) + at) = u;
+            }
+        }
+    } else {
+        for (int t = tid >> 5; t < nt; t += threads >> 5) head_norm_row(nm, Os + t * ldv, row0 + t, h, heads, dv);
+    }
+}
+
+template <int D>
+int launch_chunked(const DeltaSource& src, const DeltaNorm& nm, float* state, int num_slots, const int* seg_start, const int* seg_len,
+                   const int* state_slots, float* o, float* qp, float* M, float* N, int segments, int max_len, int heads, int dk,
+                   int dv, cudaStream_t stream) {
+    constexpr int STAGES = D == 64 ? 4 : 2, JS = D == 64 ? 4 : 2;      // (256 threads, dk tiles: JS x dk <= 256)
+    const size_t prep = (size_t)(4 * C * (dk + 4) + 2 * C * (dv + 4) + 4 * C * LDS + dk + C) * sizeof(float);
+    const size_t walk = (size_t)(STAGES * dk * (dk + 4) + (STAGES + 1 + JS) * dk * WCB) * sizeof(float);
+    const size_t outs = (size_t)(C * (dk + 4) + dk * (dv + 4) + C * (dv + 4)) * sizeof(float);
+    static bool ready = false;
+    if (!ready) {
+        constexpr int W = D ? D : 128;
+        const int most_prep = (int)((6 * C * (W + 4) + 4 * C * LDS + W + C) * sizeof(float));
+        const int most_walk = (int)((STAGES * W * (W + 4) + (STAGES + 1 + JS) * W * WCB) * sizeof(float));
+        const int most_out = (int)((2 * C * (W + 4) + W * (W + 4)) * sizeof(float));
+        if (cudaFuncSetAttribute(delta_chunk_prepare_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, most_prep) != cudaSuccess ||
+            cudaFuncSetAttribute(delta_chunk_walk_kernel<D, STAGES, JS>, cudaFuncAttributeMaxDynamicSharedMemorySize, most_walk) != cudaSuccess ||
+            cudaFuncSetAttribute(delta_chunk_out_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, most_out) != cudaSuccess)
+            return jllm_fail(JLLM_CUDA_ERROR, "delta_chunked: shared memory refused");
+        ready = true;
+    }
+    const int chunks = (max_len + C - 1) / C;
+    jllm_launch(delta_chunk_prepare_kernel<D>, dim3(chunks, heads, segments), dim3(PREP_THREADS), prep, stream, LAUNCH_DEPENDENT, src,
+                seg_start, seg_len, qp, o, M, N, heads, dk, dv);
+    if (int code = jllm_check_launch("delta_chunk_prepare")) return code;
+    jllm_launch(delta_chunk_walk_kernel<D, STAGES, JS>, dim3((dv + WCB - 1) / WCB, heads, segments), dim3(WALK_THREADS), walk, stream,
+                LAUNCH_DEPENDENT, (const float*)M, N, state, num_slots, seg_start, seg_len, state_slots, heads, dk, dv);
+    if (int code = jllm_check_launch("delta_chunk_walk")) return code;
+    jllm_launch(delta_chunk_out_kernel<D>, dim3(chunks, heads, segments), dim3(128), outs, stream, LAUNCH_DEPENDENT, (const float*)qp,
+                (const float*)N, seg_start, seg_len, o, nm, heads, dk, dv);
+    return jllm_check_launch("delta_chunk_out");
 }
 
 }  // namespace
@@ -586,17 +715,27 @@ JLLM_EXPORT int jllm_delta_tanh(const float* src, int ld, void* out, int dtype, 
 }
 
 // proj [rows, ld] float32 with r, k, a_raw (heads x dk) and v (heads x dv) at the given columns; z [rows, heads x dk] float32;
-// a_bias [heads x dk]; state [slots, heads, dk, dv] float32, read and written in place; o [rows, heads x dv] float32.
+// a_bias [heads x dk]; state [slots, heads, dk, dv] float32, read and written in place; o [rows, heads x dv] float32. With y
+// [rows, heads x dv] of type `y_dtype` (heads of at most 64 values: JLLM_UNSUPPORTED, with nothing launched, where a block does not
+// hold a head's columns) the norm and gate behind the recurrence are taken along and o is not written.
 JLLM_EXPORT int jllm_delta_recurrent(const float* proj, int ld, int r_off, int k_off, int v_off, int a_off, const float* z,
                                      const void* a_bias, int bias_dtype, float rate, float* state, int num_slots,
-                                     const int* seg_start, const int* seg_len, const int* state_slots, float* o, int segments,
-                                     int heads, int dk, int dv, cudaStream_t stream) {
+                                     const int* seg_start, const int* seg_len, const int* state_slots, float* o,
+                                     const float* gate, int ld_gate, const void* gain, int gain_dtype, float eps, void* y,
+                                     int y_dtype, int segments, int heads, int dk, int dv, cudaStream_t stream) {
     JLLM_REQUIRE(segments >= 0 && heads > 0 && heads <= 65535 && dk > 0 && dk <= 1024 && dv > 0 && dv <= 65535 * 8,
                  "delta_recurrent: segments=%d heads=%d dk=%d (at most 1024) dv=%d", segments, heads, dk, dv);
     if (segments == 0) return JLLM_OK;
     const DeltaSource src{proj, z, VecRef{a_bias, bias_dtype}, rate, ld, r_off, k_off, v_off, a_off};
+    const DeltaNorm nm{gate, y, VecRef{gain, gain_dtype}, eps, ld_gate, y_dtype};
 #define JLLM_DELTA(LS, R, CB, TOK)                                                                                             \
-    return launch_recurrent<LS, R, CB, TOK>(src, state, num_slots, seg_start, seg_len, state_slots, o, segments, heads, dk, dv, stream)
+    return launch_recurrent<LS, R, CB, TOK>(src, state, num_slots, seg_start, seg_len, state_slots, o, nm, segments, heads, dk, dv, \
+                                            stream)
+    if (y != nullptr) {
+        if (dk > 64 || dv > 64) return JLLM_UNSUPPORTED;
+        if (dv <= 32) JLLM_DELTA(4, 16, 32, 8);
+        JLLM_DELTA(4, 16, 64, 8);
+    }
     if (dk <= 32) JLLM_DELTA(4, 8, 32, 8);
     if (dk <= 64) JLLM_DELTA(4, 16, 32, 8);
     if (dk <= 128) JLLM_DELTA(8, 16, 32, 8);
@@ -606,41 +745,27 @@ JLLM_EXPORT int jllm_delta_recurrent(const float* proj, int ld, int r_off, int k
 #undef JLLM_DELTA
 }
 
-// The same for prompt portions, in chunks of 32 tokens: three launches. qp [rows, heads x dk], M [chunks, heads, dk, dk] and N
+// The same for prompt portions, in chunks of 32 tokens: three launches (the last one takes the norm and gate along with y). qp [rows, heads x dk], M [chunks, heads, dk, dk] and N
 // [chunks, heads, dk, dv] float32 scratch, chunks >= rows / 32 + segments. JLLM_UNSUPPORTED, with nothing launched, where the
 // sizes are not taken.
 JLLM_EXPORT int jllm_delta_chunked(const float* proj, int ld, int r_off, int k_off, int v_off, int a_off, const float* z,
                                    const void* a_bias, int bias_dtype, float rate, float* state, int num_slots,
                                    const int* seg_start, const int* seg_len, const int* state_slots, float* o, float* qp, float* M,
-                                   float* N, int segments, int max_len, int heads, int dk, int dv, cudaStream_t stream) {
+                                   float* N, const float* gate, int ld_gate, const void* gain, int gain_dtype, float eps,
+                                   void* y, int y_dtype, int segments, int max_len, int heads, int dk, int dv,
+                                   cudaStream_t stream) {
     if (dk % 4 || dv % 4 || dk > 128 || dv > 128 || dk <= 0 || dv <= 0 || ld % 4 || r_off % 4 || k_off % 4 || v_off % 4 || a_off % 4 ||
         ((uintptr_t)proj % 16) || ((uintptr_t)z % 16) || !(rate * C <= 60.f) || segments > 65535 || heads > 65535)
         return JLLM_UNSUPPORTED;
     if (segments <= 0 || max_len <= 0) return JLLM_OK;
     const DeltaSource src{proj, z, VecRef{a_bias, bias_dtype}, rate, ld, r_off, k_off, v_off, a_off};
-    const size_t prep = (size_t)(4 * C * (dk + 4) + 2 * C * (dv + 4) + 4 * C * LDS + dk + C) * sizeof(float);
-    const size_t walk = (size_t)(2 * dk * (dk + 4) + 3 * dk * WCB) * sizeof(float);
-    const size_t outs = (size_t)(C * (dk + 4) + dk * (dv + 4)) * sizeof(float);
-    static bool ready = false;
-    if (!ready) {
-        const int most_prep = (int)((4 * C * 132 + 2 * C * 132 + 4 * C * LDS + 128 + C) * sizeof(float));
-        const int most_walk = (int)((2 * 128 * 132 + 3 * 128 * WCB) * sizeof(float));
-        const int most_out = (int)((C * 132 + 128 * 132) * sizeof(float));
-        if (cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, most_prep) != cudaSuccess ||
-            cudaFuncSetAttribute(delta_chunk_walk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, most_walk) != cudaSuccess ||
-            cudaFuncSetAttribute(delta_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, most_out) != cudaSuccess)
-            return jllm_fail(JLLM_CUDA_ERROR, "delta_chunked: shared memory refused");
-        ready = true;
-    }
-    const int chunks = (max_len + C - 1) / C;
-    jllm_launch(delta_chunk_prepare_kernel, dim3(chunks, heads, segments), dim3(128), prep, stream, LAUNCH_DEPENDENT, src, seg_start,
-                seg_len, qp, o, M, N, heads, dk, dv);
-    if (int code = jllm_check_launch("delta_chunk_prepare")) return code;
-    const int wthreads = ((dk / 4) * (WCB / 2) + 31) / 32 * 32;
-    jllm_launch(delta_chunk_walk_kernel, dim3((dv + WCB - 1) / WCB, heads, segments), dim3(wthreads), walk, stream, LAUNCH_DEPENDENT,
-                (const float*)M, N, state, num_slots, seg_start, seg_len, state_slots, heads, dk, dv);
-    if (int code = jllm_check_launch("delta_chunk_walk")) return code;
-    jllm_launch(delta_chunk_out_kernel, dim3(chunks, heads, segments), dim3(128), outs, stream, LAUNCH_DEPENDENT, (const float*)qp,
-                (const float*)N, seg_start, seg_len, o, heads, dk, dv);
-    return jllm_check_launch("delta_chunk_out");
+    const DeltaNorm nm{gate, y, VecRef{gain, gain_dtype}, eps, ld_gate, y_dtype};
+#define JLLM_CHUNKED(D)                                                                                                        \
+    return launch_chunked<D>(src, nm, state, num_slots, seg_start, seg_len, state_slots, o, qp, M, N, segments, max_len, heads, dk, \
+                             dv, stream)
+    if (dk == 64 && dv == 64 && (y == nullptr || (ld_gate % 4 == 0 && ((uintptr_t)gate % 16) == 0 && ((uintptr_t)y % 16) == 0)))
+        JLLM_CHUNKED(64);
+    if (dk == 128 && dv == 128) JLLM_CHUNKED(128);
+    JLLM_CHUNKED(0);
+#undef JLLM_CHUNKED
 }

@@ -128,7 +128,7 @@ class _Signatures:
     jllm_bounds_error_rowwise = [P]
     jllm_set_pdl = [I]
     jllm_launch_plan = [ctypes.c_longlong, I]
-    jllm_embed_rows = [P, P, I, P, I, I, I, P]
+    jllm_embed_rows = [P, P, I, P, I, I, I, F, P]
     jllm_feed_tokens = [P, P, I, I, P]
     jllm_rmsnorm = [P, P, I, P, I, P, I, I, F, P]
     jllm_swiglu = [P, P, I, I, I, I, P]
@@ -198,18 +198,18 @@ class _Signatures:
     jllm_map_difference = [P, I, I, I, F, F, F, P, I, I, I, I, P]
     jllm_bounds_error_delta_recurrence = [P]
     jllm_delta_tanh = [P, I, P, I, I, I, P]
-    jllm_delta_recurrent = [P, I, I, I, I, I, P, P, I, F, P, I, P, P, P, P, I, I, I, I, P]
-    jllm_delta_chunked = [P, I, I, I, I, I, P, P, I, F, P, I, P, P, P, P, P, P, P, I, I, I, I, I, P]
+    jllm_delta_recurrent = [P, I, I, I, I, I, P, P, I, F, P, I, P, P, P, P, P, I, P, I, F, P, I, I, I, I, I, P]
+    jllm_delta_chunked = [P, I, I, I, I, I, P, P, I, F, P, I, P, P, P, P, P, P, P, P, I, P, I, F, P, I, I, I, I, I, I, P]
     jllm_sample = [P, I, I, I, P, P, P, P, P, P, P]
 
 
 # ---------------------------------------------------------------------------------------------------------
 
-def embed_rows(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor) -> None:
-    """out[r] = table[ids[r]] as float32; ids int32 [rows]."""
+def embed_rows(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
+    """out[r] = table[ids[r]] * scale as float32; ids int32 [rows]."""
     assert ids.dtype == torch.int32 and out.dtype == torch.float32 and table.dim() == 2
     _call("jllm_embed_rows", ids.data_ptr(), table.data_ptr(), _DT[table.dtype], out.data_ptr(), ids.numel(),
-          table.shape[1], table.shape[0], _stream())
+          table.shape[1], table.shape[0], float(scale), _stream())
 
 
 def feed_tokens(ids: torch.Tensor, sampled: torch.Tensor) -> None:
@@ -685,32 +685,47 @@ def _delta_args(proj, r_off, k_off, v_off, a_off, z, a_bias, rate, state, seg_st
             state_slots.data_ptr(), out.data_ptr())
 
 
+def _delta_norm_args(norm):
+    """norm = (gate view [rows, heads x value_dim] float32, gain [heads x value_dim], eps, y), or None."""
+    if norm is None:
+        return (0, 0, 0, F32, 0.0, 0, F32)
+    gate, gain, eps, y = norm
+    assert gate.dtype == torch.float32 and gate.stride(1) == 1 and y.is_contiguous() and y.shape == gate.shape
+    return (gate.data_ptr(), gate.stride(0), gain.data_ptr(), _DT[gain.dtype], float(eps), y.data_ptr(), _DT[y.dtype])
+
+
 def delta_recurrent(proj, r_off, k_off, v_off, a_off, z, a_bias, rate, state, seg_start, seg_len, state_slots, out, heads, key_dim,
-                    value_dim) -> None:
+                    value_dim, norm=None) -> bool:
     """The generalized delta rule token by token: per (segment, head), with u = k / sqrt(sum(k^2) + 1e-6), d = exp(-rate
     sigmoid(z)), a = sigmoid(a_raw + a_bias): S = diag(d) S - (a u) (u^T S) + k v^T, o = S^T r. proj float32 [rows, *]: r, k, a_raw
     (heads x key_dim) and v (heads x value_dim) at the given columns; z float32 [rows, heads x key_dim]; state [slots, heads,
-    key_dim, value_dim] float32, read and written in place; out float32 [rows, heads x value_dim]."""
+    key_dim, value_dim] float32, read and written in place; out float32 [rows, heads x value_dim]. With `norm` = (gate, gain, eps, y)
+    the same launch makes y = rms(o) per head * gain * sigmoid(gate) instead of out; it says False, having launched nothing, for
+    heads that a block does not hold as a whole (more than 64 values)."""
+    if norm is not None and (key_dim > 64 or value_dim > 64):
+        return False
     _call("jllm_delta_recurrent", *_delta_args(proj, r_off, k_off, v_off, a_off, z, a_bias, rate, state, seg_start, seg_len,
-                                               state_slots, out), seg_start.numel(), heads, key_dim, value_dim, _stream())
+                                               state_slots, out), *_delta_norm_args(norm), seg_start.numel(), heads, key_dim,
+          value_dim, _stream())
+    return True
 
 
 DELTA_CHUNK = 32      # tokens of a chunk (C in delta_recurrence.cu)
 
 
 def delta_chunked(proj, r_off, k_off, v_off, a_off, z, a_bias, rate, state, seg_start, seg_len, state_slots, out, heads, key_dim,
-                  value_dim, max_len, qp, transition, added) -> bool:
+                  value_dim, max_len, qp, transition, added, norm=None) -> bool:
     """`delta_recurrent` for prompt portions, in chunks of 32 tokens (all float32; only the grouping of sums differs): three
-    launches. `max_len`: the longest segment's rows. qp [rows, heads x key_dim], transition [chunks, heads x key_dim x key_dim] and
-    added [chunks, heads x key_dim x value_dim] float32 scratch, chunks >= rows / 32 + segments. Says False, having launched
-    nothing, where the sizes are not taken."""
+    launches, the last of which takes the norm and gate along with `norm`. `max_len`: the longest segment's rows. qp [rows, heads
+    x key_dim], transition [chunks, heads x key_dim x key_dim] and added [chunks, heads x key_dim x value_dim] float32 scratch, chunks
+    >= rows / 32 + segments. Says False, having launched nothing, where the sizes are not taken."""
     S = seg_start.numel()
     assert qp.dtype == transition.dtype == added.dtype == torch.float32 and qp.is_contiguous()
     if proj.shape[0] // DELTA_CHUNK + S > transition.shape[0]:
         return False
     code = library().jllm_delta_chunked(*_delta_args(proj, r_off, k_off, v_off, a_off, z, a_bias, rate, state, seg_start, seg_len,
-                                                     state_slots, out), qp.data_ptr(), transition.data_ptr(), added.data_ptr(), S,
-                                        int(max_len), heads, key_dim, value_dim, _stream())
+                                                     state_slots, out), qp.data_ptr(), transition.data_ptr(), added.data_ptr(),
+                                        *_delta_norm_args(norm), S, int(max_len), heads, key_dim, value_dim, _stream())
     if code == 3:        # the library's word for "these sizes are not taken"
         return False
     if code != 0:

@@ -324,21 +324,43 @@ template <int V> __device__ __forceinline__ void store_pack(__nv_bfloat16* p, co
     }
 }
 
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
 constexpr int CONV_TAPS = 16;     // most taps
 constexpr int CONV_RUN = 8;       // rows of a block in a step with prompt portions
 
 // RUN rows a block; `single` (RUN = 1): every segment is one row, and the state is brought up to date here. V channels a thread
-// at a time.
-template <typename Tout, int RUN, int V>
+// at a time. TAPS > 0: the number of taps, known to the compiler: the taps' weights and the window of normed rows stay in
+// registers from row to row; 0: read from the argument, every row fetched anew.
+template <typename Tout, int RUN, int V, int TAPS>
 __global__ void __launch_bounds__(256)
 norm_conv_kernel(const float* __restrict__ x, VecRef gain, VecRef conv, float* __restrict__ state, int num_slots,
                  const int* __restrict__ row_seg, const int* __restrict__ seg_start, const int* __restrict__ state_slots,
-                 Tout* __restrict__ out, int rows, int dim, int taps, float eps, int single) {
+                 Tout* __restrict__ out, int rows, int dim, int taps_arg, float eps, int single) {
     __shared__ float inv[RUN + CONV_TAPS];
     __shared__ float scratch[33];
+    __shared__ int where[RUN][2];          // a row's place in its segment, and its state slot (-1: none that may be touched)
+    const int taps = TAPS ? TAPS : taps_arg;
+    if constexpr (RUN == 1) {
+        // what this row will read besides x is older than the kernel in front of this one (weights, the step's tables, a state
+        // that an earlier step left): on its way into L2 while that kernel still runs
+        const int slot = state_slots[row_seg[blockIdx.x]];
+        if (single && jllm_in_bounds(slot, num_slots, BOUNDS_SLOT)) {
+            const char* st = reinterpret_cast<const char*>(state + (size_t)slot * (taps - 1) * dim);
+            for (long long e = threadIdx.x * 128ll; e < (long long)(taps - 1) * dim * 4; e += 256 * 128) prefetch_l2(st + e);
+            const char* cv = static_cast<const char*>(conv.p);
+            const long long bytes = (long long)taps * dim * (conv.dtype == JLLM_F32 ? 4 : 2);
+            for (long long e = threadIdx.x * 128ll; e < bytes; e += 256 * 128) prefetch_l2(cv + e);
+        }
+    }
     pdl_wait();
     pdl_trigger();
     const int r0 = blockIdx.x * RUN, r1 = min(rows, r0 + RUN), lo = single ? r0 : max(0, r0 - (taps - 1));
+    if (threadIdx.x < r1 - r0) {
+        const int seg = row_seg[r0 + threadIdx.x], slot = state_slots[seg];
+        where[threadIdx.x][0] = single ? 0 : r0 + threadIdx.x - seg_start[seg];
+        where[threadIdx.x][1] = jllm_in_bounds(slot, num_slots, BOUNDS_SLOT) ? slot : -1;
+    }
     if constexpr (RUN == 1) {
         // (one row: all of the block's threads on it; in a step with portions RUN is larger)
         float ss = 0.f;
@@ -364,28 +386,55 @@ norm_conv_kernel(const float* __restrict__ x, VecRef gain, VecRef conv, float* _
             for (int k = 0; k < V; ++k) h.v[k] = __fmul_rn(__fmul_rn(h.v[k], f), g[k]);
             return h;
         };
-        for (int r = r0; r < r1; ++r) {
-            const int seg = row_seg[r], slot = state_slots[seg], t = single ? 0 : r - seg_start[seg];
-            const bool ok = jllm_in_bounds(slot, num_slots, BOUNDS_SLOT);
-            float* st = state + (size_t)(ok ? slot : 0) * max(taps - 1, 1) * dim + i;
-            const Pack<V> h = normed(r);
-            Pack<V> acc = h;
-            for (int j = 0; j < taps; ++j) {
-                const int at = t - (taps - 1) + j;
-                Pack<V> in;
-                if (j == taps - 1) in = h;
-                else if (at >= 0) in = normed(r - (taps - 1) + j);
-                else if (ok) in = load_pack<V>(st + (size_t)(taps - 1 + at) * dim);
-                else {
+        // the input of tap j of row r, which lies at place t of its segment: an earlier row, or what the state holds
+        auto earlier = [&](int r, int t, int slot, int j) {
+            const int at = t - (taps - 1) + j;
+            if (at >= 0) return normed(r - (taps - 1) + j);
+            Pack<V> in = {};
+            if (slot >= 0) in = load_pack<V>(state + ((size_t)slot * (taps - 1) + taps - 1 + at) * dim + i);
+            return in;
+        };
+        if constexpr (TAPS > 0) {
+            float w[TAPS][V];
 #pragma unroll
-                    for (int k = 0; k < V; ++k) in.v[k] = 0.f;
+            for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+                for (int k = 0; k < V; ++k) w[j][k] = conv[(i + k) * TAPS + j];
+            Pack<V> win[TAPS];
+            for (int r = r0; r < r1; ++r) {
+                const int t = where[r - r0][0], slot = where[r - r0][1];
+                if (r == r0 || t == 0) {
+#pragma unroll
+                    for (int j = 0; j + 1 < TAPS; ++j) win[j] = earlier(r, t, slot, j);
                 }
+                win[TAPS - 1] = normed(r);
+                Pack<V> acc = win[TAPS - 1];
 #pragma unroll
-                for (int k = 0; k < V; ++k) acc.v[k] = fmaf(conv[(i + k) * taps + j], in.v[k], acc.v[k]);
-                // a step of single rows: this thread alone touches these channels of the slot; entry j - 1 has been read
-                if (single && j > 0 && ok) store_pack<V>(st + (size_t)(j - 1) * dim, in);
+                for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+                    for (int k = 0; k < V; ++k) acc.v[k] = fmaf(w[j][k], win[j].v[k], acc.v[k]);
+                store_pack<V>(out + (size_t)r * dim + i, acc);
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; ++j) win[j] = win[j + 1];
+                if (single && slot >= 0) {      // (this thread alone touches these channels of the slot)
+#pragma unroll
+                    for (int j = 0; j + 1 < TAPS; ++j) store_pack<V>(state + ((size_t)slot * (TAPS - 1) + j) * dim + i, win[j]);
+                }
             }
-            store_pack<V>(out + (size_t)r * dim + i, acc);
+        } else {
+            for (int r = r0; r < r1; ++r) {
+                const int t = where[r - r0][0], slot = where[r - r0][1];
+                const Pack<V> h = normed(r);
+                Pack<V> acc = h;
+                for (int j = 0; j < taps; ++j) {
+                    const Pack<V> in = j == taps - 1 ? h : earlier(r, t, slot, j);
+#pragma unroll
+                    for (int k = 0; k < V; ++k) acc.v[k] = fmaf(conv[(i + k) * taps + j], in.v[k], acc.v[k]);
+                    // a step of single rows: entry j - 1 of the slot has been read by its only reader
+                    if (single && j > 0 && slot >= 0) store_pack<V>(state + ((size_t)slot * (taps - 1) + j - 1) * dim + i, in);
+                }
+                store_pack<V>(out + (size_t)r * dim + i, acc);
+            }
         }
     }
 }
@@ -404,7 +453,7 @@ norm_conv_save_kernel(const float* __restrict__ x, VecRef gain, float* __restric
     const int lo = max(0, n - (taps - 1));
     rms_factors(x, first + lo, first + n, dim, eps, inv);
     __syncthreads();
-    for (int i = threadIdx.x; i < dim; i += blockDim.x)
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < dim; i += gridDim.y * blockDim.x)
         for (int j = 0; j + 1 < taps; ++j) {        // (ascending: the old entry j + n is read before it is written)
             const int at = n - (taps - 1) + j;
             st[(size_t)j * dim + i] = at >= 0 ? __fmul_rn(__fmul_rn(x[(size_t)(first + at) * dim + i], inv[at - lo]), gain[i])
@@ -524,22 +573,30 @@ JLLM_EXPORT int jllm_norm_conv(const float* x, const void* gain, int gain_dtype,
     if (rows == 0) return JLLM_OK;
     const VecRef g{gain, gain_dtype}, c{conv, conv_dtype};
     const bool vec = dim % 4 == 0 && (((uintptr_t)x | (uintptr_t)state | (uintptr_t)out) % 16) == 0;
-#define JLLM_NORM_CONV(T, RUN, V)                                                                                              \
-    jllm_launch(norm_conv_kernel<T, RUN, V>, dim3((rows + RUN - 1) / RUN), dim3(256), 0, stream, LAUNCH_DEPENDENT, x, g, c, state,  \
-                num_slots, row_seg, seg_start, state_slots, (T*)out, rows, dim, taps, eps, single)
+#define JLLM_NORM_CONV(T, RUN, V, TAPS)                                                                                        \
+    jllm_launch(norm_conv_kernel<T, RUN, V, TAPS>, dim3((rows + RUN - 1) / RUN), dim3(256), 0, stream, LAUNCH_DEPENDENT, x, g, c,   \
+                state, num_slots, row_seg, seg_start, state_slots, (T*)out, rows, dim, taps, eps, single)
+#define JLLM_NORM_CONV_TAPS(T, RUN, V)                                                                                         \
+    do {                                                                                                                       \
+        if (taps == 2) JLLM_NORM_CONV(T, RUN, V, 2);                                                                           \
+        else if (taps == 3) JLLM_NORM_CONV(T, RUN, V, 3);                                                                      \
+        else if (taps == 4) JLLM_NORM_CONV(T, RUN, V, 4);                                                                      \
+        else JLLM_NORM_CONV(T, RUN, V, 0);                                                                                     \
+    } while (0)
 #define JLLM_NORM_CONV_T(T)                                                                                                    \
     do {                                                                                                                       \
-        if (single && vec) JLLM_NORM_CONV(T, 1, 4);                                                                            \
-        else if (single) JLLM_NORM_CONV(T, 1, 1);                                                                              \
-        else if (vec) JLLM_NORM_CONV(T, CONV_RUN, 4);                                                                          \
-        else JLLM_NORM_CONV(T, CONV_RUN, 1);                                                                                   \
+        if (single && vec) JLLM_NORM_CONV_TAPS(T, 1, 4);                                                                       \
+        else if (single) JLLM_NORM_CONV_TAPS(T, 1, 1);                                                                         \
+        else if (vec) JLLM_NORM_CONV_TAPS(T, CONV_RUN, 4);                                                                     \
+        else JLLM_NORM_CONV_TAPS(T, CONV_RUN, 1);                                                                              \
     } while (0)
     if (out_dtype == JLLM_F32) JLLM_NORM_CONV_T(float);
     else JLLM_NORM_CONV_T(__nv_bfloat16);
 #undef JLLM_NORM_CONV_T
+#undef JLLM_NORM_CONV_TAPS
 #undef JLLM_NORM_CONV
     if (!single && taps > 1)
-        jllm_launch(norm_conv_save_kernel, dim3(segments), dim3(256), 0, stream, LAUNCH_DEPENDENT, x, g, state, num_slots, seg_start,
+        jllm_launch(norm_conv_save_kernel, dim3(segments, max(1, min(16, (dim + 255) / 256))), dim3(256), 0, stream, LAUNCH_DEPENDENT, x, g, state, num_slots, seg_start,
                     seg_len, state_slots, dim, taps, eps);
     return jllm_check_launch("norm_conv");
 }

@@ -8,30 +8,40 @@
 #include "head_rotate.cuh"
 
 // ---------------------------------------------------------------------------------------------------
-// x[r, :] = table[ids[r], :]  (float residual stream from a float or bfloat16 table)
+// x[r, :] = table[ids[r], :] * scale  (float residual stream from a float or bfloat16 table)
 // ---------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x,
-                                  int dim, int vocab) {
+                                  int dim, int vocab, float scale) {
     const int r = blockIdx.x;
     int id = ids[r];
     jllm_in_bounds(id, vocab, BOUNDS_TOKEN);           // checked build: recorded
     id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);  // ids are validated on the host; never read out of bounds
     const T* src = table + (size_t)id * dim;
     float* dst = x + (size_t)r * dim;
-    for (int i = threadIdx.x; i < dim; i += blockDim.x) dst[i] = to_float(src[i]);
+    if ((dim & 3) == 0 && (((uintptr_t)table | (uintptr_t)x) & 15u) == 0) {      // four values a thread at a time
+        for (int i = threadIdx.x * 4; i < dim; i += blockDim.x * 4) {
+            alignas(16) T v[4];
+            if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(v) = *reinterpret_cast<const uint2*>(src + i);
+            else *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(src + i);
+            *reinterpret_cast<float4*>(dst + i) = make_float4(__fmul_rn(to_float(v[0]), scale), __fmul_rn(to_float(v[1]), scale),
+                                                              __fmul_rn(to_float(v[2]), scale), __fmul_rn(to_float(v[3]), scale));
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < dim; i += blockDim.x) dst[i] = __fmul_rn(to_float(src[i]), scale);
 }
 
 JLLM_BOUNDS_READER(rowwise)
 
 JLLM_EXPORT int jllm_embed_rows(const int* ids, const void* table, int table_dtype, float* x, int rows, int dim,
-                                int vocab, cudaStream_t stream) {
+                                int vocab, float scale, cudaStream_t stream) {
     JLLM_REQUIRE(rows >= 0 && dim > 0 && vocab > 0, "embed_rows: rows=%d dim=%d vocab=%d", rows, dim, vocab);
     if (rows == 0) return JLLM_OK;
     if (table_dtype == JLLM_F32)
-        embed_rows_kernel<float><<<rows, 256, 0, stream>>>(ids, (const float*)table, x, dim, vocab);
+        embed_rows_kernel<float><<<rows, 256, 0, stream>>>(ids, (const float*)table, x, dim, vocab, scale);
     else
-        embed_rows_kernel<__nv_bfloat16><<<rows, 256, 0, stream>>>(ids, (const __nv_bfloat16*)table, x, dim, vocab);
+        embed_rows_kernel<__nv_bfloat16><<<rows, 256, 0, stream>>>(ids, (const __nv_bfloat16*)table, x, dim, vocab, scale);
     return jllm_check_launch("embed_rows");
 }
 

@@ -153,9 +153,7 @@ class DecoderModel:
             x = stack[0]
         else:
             x = self.rt.buffer("residual", self.dim, torch.float32)[:rows]
-        ops.embed_rows(batch.token_ids, self.embedding, x)
-        if self.embedding_scale != 1.0:
-            ops.scale_values(x, self.embedding_scale)
+        ops.embed_rows(batch.token_ids, self.embedding, x, self.embedding_scale)
         for pe in self.position_encodings:
             pe.on_embedding(x, batch)
         for i, run in enumerate(schedule):

@@ -13,7 +13,8 @@ besides the projections (decays, removal rates, unit keys) is 32-bit in both pre
 product leaves in float32 too. The state S [heads, dk, dv] is float32 and lives in the cache manager's state slots (zero when a
 request is opened). Single rows run token by token (`ops.delta_recurrent`), prompt portions in chunks of 32 tokens
 (`ops.delta_chunked`: within a chunk the removals are the solution of a triangular system that is linear in the state in front
-of it); a step of both runs each on its own rows.
+of it); a step of both runs each on its own rows. The norm and gate behind the recurrence ride in its last launch (single rows:
+for heads of up to 64 values, else in a launch of their own).
 """
 from __future__ import annotations
 
@@ -72,8 +73,8 @@ class GeneralDelta(Mixer):
     def decode_bucket_cap(self, rows: int) -> int:
         return 1                       # nothing here looks at the context's length
 
-    def _chunks(self, proj, z, batch, state, o, segments: int, rows: int) -> bool:
-        """Rows [0, rows), segments [0, segments) in chunks; False where the sizes are not taken."""
+    def _chunks(self, proj, z, batch, state, o, segments: int, rows: int, gate, y) -> bool:
+        """Rows [0, rows), segments [0, segments) in chunks, their norm and gate included; False where the sizes are not taken."""
         s = self.spec
         H, dk, dv = s.heads, s.key_dim, s.value_dim
         r_off, k_off, v_off, _, a_off, _ = self.offsets
@@ -83,7 +84,7 @@ class GeneralDelta(Mixer):
         added = self.rt.buffer("delta_chunk_added", H * dk * dv, torch.float32, rows=room)
         return ops.delta_chunked(proj[:rows], r_off, k_off, v_off, a_off, z[:rows], self.a_bias, s.decay_rate, state,
                                  batch.seg_start[:segments], batch.seg_len[:segments], batch.state_slots[:segments], o[:rows], H, dk,
-                                 dv, batch.max_q_len, qp, transition, added)
+                                 dv, batch.max_q_len, qp, transition, added, norm=(gate[:rows], self.gain, s.norm_eps, y[:rows]))
 
     def forward(self, xb, x, batch, cache) -> None:
         s, rows = self.spec, xb.shape[0]
@@ -98,17 +99,21 @@ class GeneralDelta(Mixer):
         z = self.rt.buffer("delta_decay_logits", H * dk, torch.float32)[:rows]
         self.decay.forward(t, z)
         o = self.rt.buffer("delta_out", H * dv, torch.float32)[:rows]
-        segments, done = batch.seg_start.numel(), 0            # segments whose rows have run
+        y = self.rt.buffer("delta_gated", H * dv)[:rows]
+        gate = proj[:, g_off:g_off + H * dv]
+        segments, done, done_rows = batch.seg_start.numel(), 0, 0         # segments (rows) that have run
         if not batch.decode_only:
             # prompt portions in chunks; the single rows beside them (the scheduler puts them last) token by token
             ms, mr = (batch.multi_segments, batch.multi_rows) if batch.multi_segments >= 0 else (segments, rows)
-            if ms > 0 and self._chunks(proj, z, batch, cache.state, o, ms, mr):
-                done = ms
+            if ms > 0 and self._chunks(proj, z, batch, cache.state, o, ms, mr, gate, y):
+                done, done_rows = ms, mr
         if done < segments:
-            ops.delta_recurrent(proj, r_off, k_off, v_off, a_off, z, self.a_bias, s.decay_rate, cache.state, batch.seg_start[done:],
-                                batch.seg_len[done:], batch.state_slots[done:], o, H, dk, dv)
-        y = self.rt.buffer("delta_gated", H * dv)[:rows]
-        ops.gated_head_norm(o, proj[:, g_off:g_off + H * dv], self.gain, s.norm_eps, 1.0, y, H, dv, "sigmoid", gain_per_column=True)
+            args = (proj, r_off, k_off, v_off, a_off, z, self.a_bias, s.decay_rate, cache.state, batch.seg_start[done:],
+                    batch.seg_len[done:], batch.state_slots[done:], o, H, dk, dv)
+            if not ops.delta_recurrent(*args, norm=(gate, self.gain, s.norm_eps, y)):
+                ops.delta_recurrent(*args)
+                ops.gated_head_norm(o[done_rows:], gate[done_rows:], self.gain, s.norm_eps, 1.0, y[done_rows:], H, dv, "sigmoid",
+                                    gain_per_column=True)
         self.out.forward(y, x, accumulate=not self.overwrite)
 
 
