@@ -87,8 +87,11 @@ def input_convolution(h, conv):
     return out
 
 
-def delta_recurrence(r, k, v, d, a):
-    """r, k, v, d, a [T, heads, dim] -> o [T, heads, dim]; the state starts at zero."""
+def delta_recurrence(r, k, v, d, a, turns_out=None):
+    """r, k, v, d, a [T, heads, dim] -> o [T, heads, dim]; the state starts at zero. `turns_out` (a list) gets one tensor [T]: the
+    least |o| / (|S| |r|) of a token's heads. Near 0 the direction of o, all that the norm behind it keeps, hangs on the last bits
+    of its inputs: a sequence's first token has S = k v^T and o = (k . r) v, whose SIGN is that of k . r."""
+    near = torch.ones(k.shape[0], dtype=k.dtype)
     T, H, n = k.shape
     S = torch.zeros((H, n, v.shape[2]), dtype=k.dtype)
     o = torch.zeros_like(v)
@@ -97,16 +100,19 @@ def delta_recurrence(r, k, v, d, a):
         read = torch.einsum("hi,hij->hj", u, S)
         S = d[t][:, :, None] * S - (a[t] * u)[:, :, None] * read[:, None, :] + k[t][:, :, None] * v[t][:, None, :]
         o[t] = torch.einsum("hij,hi->hj", S, r[t])
+        near[t] = (o[t].norm(dim=-1) / (S.flatten(1).norm(dim=-1) * r[t].norm(dim=-1) + 1e-300)).min()
+    if turns_out is not None:
+        turns_out.append(near)
     return o
 
 
-def general_delta(h, w, p, m, eps):
+def general_delta(h, w, p, m, eps, turns_out=None):
     T, H, n = h.shape[0], int(m["heads"]), int(m["dim"])
     r, k, v = ((h @ w[p + x].T).view(T, H, n) for x in ("r", "k", "v"))
     decay = torch.sigmoid(torch.tanh(h @ w[p + "w1"].T) @ w[p + "w2"].T + w[p + "w0"])
     d = torch.exp(-math.exp(-0.5) * decay).view(T, H, n)
     a = torch.sigmoid(h @ w[p + "a"].T + w[p + "a.b"]).view(T, H, n)
-    o = rms(delta_recurrence(r, k, v, d, a), eps).reshape(T, H * n)
+    o = rms(delta_recurrence(r, k, v, d, a, turns_out), eps).reshape(T, H * n)
     return (o * w[p + "norm"] * torch.sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
 
 
@@ -186,16 +192,17 @@ def feed_forward(h, w, p):
 
 # ---- the model ------------------------------------------------------------------------------------------------------
 
-def forward(cfg, w, tokens, layers_out=None):
-    """Logits [T, vocab] of one whole sequence; `layers_out` (a list) gets the residual stream after every layer."""
-    x = w["embed"][torch.tensor(tokens)] * float(cfg["embedding"]["scale"])
+def forward(cfg, w, tokens, layers_out=None, turns_out=None):
+    """Logits [T, vocab] of one whole sequence; `layers_out` (a list) gets the residual stream after every layer, `turns_out` (a
+    list) one tensor [T] per delta layer: how near a head's result is to turning its sign (see `delta_recurrence`)."""
+    x = w["embed"][torch.tensor(tokens)] * float(cfg.get("embedding", {}).get("scale", 1.0))
     eps = float(cfg["norm"]["eps"])
     kept = {}                                     # layer -> the keys and values it would cache
     for i, layer in enumerate(cfg["layers"]):
         p, m = f"l{i}.", layer["mixer"]
         h = input_convolution(norm(x, w[p + "norm1"], eps), w[p + "canon1"])
         if layer["type"] == "general_delta":
-            y = general_delta(h, w, p + "mix.", m, eps)
+            y = general_delta(h, w, p + "mix.", m, eps, turns_out)
         elif layer["type"] == "attention":
             if m.get("kv_from") is None:
                 kept[i] = differential_keys_values(h, w, p + "mix.", m)
