@@ -12,6 +12,7 @@ from .movivik import parse_movivik
 from .bozevik import parse_bozevik
 from .guvolix import parse_guvolix
 from .fusazen import parse_fusazen
+from .narolorn import parse_narolorn
 
 register_architecture("qwen3", parse_qwen3, replace=True)
 register_architecture("Madevik", parse_madevik, replace=True)
@@ -19,3 +20,4 @@ register_architecture("Movivik", parse_movivik, replace=True)
 register_architecture("Bozevik", parse_bozevik, replace=True)
 register_architecture("Guvolix", parse_guvolix, replace=True)
 register_architecture("Fusazen", parse_fusazen, replace=True)
+register_architecture("Narolorn", parse_narolorn, replace=True)

@@ -72,6 +72,12 @@ class MixerSpec:
     kind: str = field(default="", init=False)
 
 
+def tile_width(w: int) -> int:
+    """The width (64, 128 or 256 values) that the attention tile kernels take and that rows of `w` values are filled up to where
+    that adds at most a third; 0 where none is near."""
+    return next((tile for tile in (64, 128, 256) if w <= tile <= w + w // 3), 0)
+
+
 @dataclass(frozen=True)
 class AttentionNames:
     """Checkpoint names of an attention's tensors, relative to the mixer's prefix."""
@@ -101,7 +107,9 @@ class GqaAttentionSpec(MixerSpec):
     attention (`maps` = 2): every head's query and key are two maps [map 1, map 2] of head_dim values each, both attend the same
     values, and with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff the head's result is rms(a1 - lambda a2) (1 - diff). A
     mixer with `own_kv` False has no key and value projections: it reads the rows that another run cached (the schedule's
-    `cache_of`), with its own queries and mask."""
+    `cache_of`), with its own queries and mask. Scores may be capped (`softcap`: s = softcap tanh(scale (q . k) / softcap)), the
+    queries may grow with their position (`temp_every` > 0: times 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)), and the values
+    may be the keys as projected, before norm and rotation (`keys_as_values`: there is no value projection)."""
     kind: str = field(default="gqa_attention", init=False)
     heads: int = 0
     kv_heads: int = 0
@@ -128,6 +136,10 @@ class GqaAttentionSpec(MixerSpec):
     diff: float = 0.0                      # its constant
     diff_norm_eps: float = 1e-6            # eps of the norm over a head's difference
     own_kv: bool = True                    # False: no key and value projections, another run's cache
+    softcap: float = 0.0                   # 0 = none
+    temp_every: int = 0                    # 0 = none
+    temp_coef: float = 0.0
+    keys_as_values: bool = False
 
     def __post_init__(self):
         if self.heads <= 0:
@@ -149,10 +161,14 @@ class GqaAttentionSpec(MixerSpec):
             raise ConfigError(f"attention: keep_first={self.keep_first} must not be negative and needs a window")
         if self.qk_norm_over not in ("head", "all") or self.maps not in (1, 2):
             raise ConfigError(f"attention: qk_norm_over={self.qk_norm_over!r} maps={self.maps} is not built")
+        if self.softcap < 0 or self.temp_every < 0:
+            raise ConfigError(f"attention: softcap={self.softcap} and temp_every={self.temp_every} must not be negative")
+        if self.keys_as_values and (self.v_dim != self.head_dim or self.maps != 1):
+            raise ConfigError(f"attention: values that are the keys have the keys' width {self.head_dim}, not {self.v_dim}, and one map")
         if self.wide and (self.bias or self.out_bias or self.gate != "none" or self.sink or self.unit_qk
                           or (self.qk_norm and self.qk_norm_over == "head")):
-            raise ConfigError("attention: two maps per head, norms over all heads and a factor per head are not built together "
-                              "with biases, gates, sinks, unit queries or norms per head")
+            raise ConfigError("attention: two maps per head, norms over all heads, a factor per head, growing queries and keys as values "
+                              "are not built together with biases, gates, sinks, unit queries or norms per head")
 
     @property
     def v_dim(self) -> int:
@@ -161,7 +177,8 @@ class GqaAttentionSpec(MixerSpec):
     @property
     def wide(self) -> bool:
         """Whether the rows are prepared by the kernel that lays a head's maps side by side in rows of `row_dim` values."""
-        return self.maps > 1 or self.head_scale or not self.own_kv or (self.qk_norm and self.qk_norm_over == "all")
+        return (self.maps > 1 or self.head_scale or not self.own_kv or self.temp_every > 0 or self.keys_as_values
+                or (self.qk_norm and self.qk_norm_over == "all"))
 
     @property
     def row_dim(self) -> int:
@@ -170,9 +187,8 @@ class GqaAttentionSpec(MixerSpec):
         if not self.wide:
             return max(self.head_dim, self.v_dim)
         w = max(self.maps * self.head_dim, self.v_dim)
-        for tile in (64, 128, 256):
-            if w <= tile <= w + w // 3:
-                return tile
+        if tile_width(w):
+            return tile_width(w)
         return -(-w // 16) * 16 if w <= 256 else -(-w // 8) * 8
 
 
@@ -358,7 +374,9 @@ class LatentAttentionSpec(MixerSpec):
     a rotated key part of `rope_dim` values that all heads share, cached beside the latent (the down projection then has
     rank + rope_dim rows, the last rope_dim are not normed; a query head is [key_dim values, then rope_dim rotated values]
     and its score is the sum of both dot products); and a run that makes no latent of its own but reads the rows another
-    run cached (`own_latent` False: no down projection; the schedule's `cache_of` names the run)."""
+    run cached (`own_latent` False: no down projection; the schedule's `cache_of` names the run).
+    `gate_full`: the gate has one value per value of the concatenated heads (Wg has heads x value_dim rows). `tile_rows`: cached
+    rows are filled up with zeros to a width the attention tile kernels take where that adds at most a third."""
     kind: str = field(default="latent_attention", init=False)
     heads: int = 0
     key_dim: int = 0
@@ -372,6 +390,8 @@ class LatentAttentionSpec(MixerSpec):
     rope_dim: int = 0                      # 0: nothing rotates; else the width of the shared rotated key part
     rope_table: int = -1                   # index into Decoder.rope_tables (its rotary_dim <= rope_dim values are rotated)
     own_latent: bool = True                # False: the run reads another run's cached rows and has no down projection
+    gate_full: bool = False
+    tile_rows: bool = False
 
     def __post_init__(self):
         for name in ("heads", "key_dim", "value_dim", "rank"):
@@ -381,11 +401,18 @@ class LatentAttentionSpec(MixerSpec):
             raise ConfigError(f"latent attention: q_rank={self.query_rank} and rot_dim={self.rope_dim} must not be negative")
         if (self.rope_dim > 0) != (self.rope_table >= 0):
             raise ConfigError("latent attention: a rotated key part needs a rotary table, and a table a rotated part")
+        if self.window < 0:
+            raise ConfigError(f"latent attention: window={self.window} must not be negative")
+        if (self.gate_full or self.tile_rows) and (self.query_rank or self.rope_dim or not self.own_latent):
+            raise ConfigError("latent attention: a gate of full width and filled-up rows are not built together with a query latent, "
+                              "a rotated key part or a borrowed cache")
+        if self.gate_full and not self.gated:
+            raise ConfigError("latent attention: gate_full says how wide the gate of a gated attention is")
 
     @property
     def cache_dim(self) -> int:
-        """Values of a cached row: the latent and, behind it, the rotated key part."""
-        return self.rank + self.rope_dim
+        """Values of a cached row: the latent and, behind it, the rotated key part (or zeros up to a tile's width)."""
+        return (self.tile_rows and tile_width(self.rank)) or self.rank + self.rope_dim
 
 
 @dataclass(frozen=True)
@@ -438,7 +465,9 @@ class RoutedExpertsSpec(FeedForwardSpec):
     `shared`: a dense gated feed-forward (tensors under `shared.`) that every token runs, added to the experts' sum; with
     `shared_gate` (the name, under the feed-forward's prefix, of a [1, dim] matrix Wsg) it is first multiplied by sigmoid(Wsg h),
     one number per token. `score` "softmax": s = softmax(Wr h) over all of the router's entries. `identity`: the router has
-    that many entries more than there are experts; one of them, when chosen, gives the token's input itself times its weight."""
+    that many entries more than there are experts; one of them, when chosen, gives the token's input itself times its weight.
+    `router_bias` (the name, under the feed-forward's prefix, of a vector): s is made from Wr h + bias. Softmax scores that are
+    normalized are the softmax over the chosen logits alone."""
     kind: str = field(default="routed_experts", init=False)
     experts: int = 0
     top: int = 0
@@ -453,6 +482,7 @@ class RoutedExpertsSpec(FeedForwardSpec):
     score: str = "sigmoid"                 # sigmoid | softmax
     identity: int = 0
     shared_gate: str = ""
+    router_bias: str = ""
 
     def __post_init__(self):
         if self.experts <= 0 or self.hidden <= 0:
@@ -485,6 +515,8 @@ class LayerNames:
     feed_forward_norm: str = "post_attention_layernorm."
     mixer_post_norm: str = ""              # the `sandwich_norm` arrangement: the norm behind the mixer
     feed_forward_post_norm: str = ""       # and the one behind the feed-forward
+    mixer_streams: str = "hc1."            # the `hyper_connections` arrangement: what the mixer reads of the streams and gives them
+    feed_forward_streams: str = "hc2."     # back (<name>in [S], <name>out [S], <name>mix [S, S]), and the feed-forward
 
 
 @dataclass(frozen=True)
@@ -507,6 +539,8 @@ class LayerSpec:
                                            # sandwich_norm: x += post(mixer(norm(x))); x += post'(ffn(norm'(x)))
                                            # post_norm: x += norm(mixer(x)); x += norm'(ffn(x)): the parts read x itself
                                            # parallel_residual: h = norm(x); x += mixer(h) + ffn(h): one norm feeds both parts
+                                           # hyper_connections: Core.streams copies X_s of the stream; per part y = part(norm(sum_s
+                                           # in[s] X_s)), X_t = sum_s mix[s, t] X_s + out[t] y
     names: LayerNames = LayerNames()
     residual_scale: float = 1.0
     prefix: Optional[str] = None           # the layer's checkpoint prefix where it is not ModelNames.layer.format(index)
@@ -516,6 +550,7 @@ class LayerSpec:
                                            # mixer reads h_t + sum_j c[:, j] h_(t - taps + 1 + j), h the normed rows, zeros in
                                            # front of the sequence (`pre_norm` arrangement)
     input_conv_taps: int = 0
+    streams: int = 0                       # `hyper_connections`: the model's Core.streams
 
 
 @dataclass(frozen=True)
@@ -542,6 +577,8 @@ class Core:
     description: str = ""
     logit_scale: float = 1.0               # the head's result is multiplied by it
     embedding_scale: float = 1.0           # the embedded rows are multiplied by it
+    logit_softcap: float = 0.0             # c > 0: the head's result z becomes c tanh(z / c)
+    streams: int = 0                       # > 0: a residual of that many streams (every layer arranges `hyper_connections`)
 
 
 @dataclass(frozen=True)
@@ -561,6 +598,11 @@ class Decoder:
             raise ConfigError(f"num_hidden_layers={self.core.layers} but {len(self.layers)} layer specs")
         if not self.schedule:
             object.__setattr__(self, "schedule", tuple(LayerRun(l) for l in range(len(self.layers))))
+        if any((l.arrangement == "hyper_connections") != (self.core.streams > 0) or l.streams != self.core.streams for l in self.layers):
+            raise ConfigError(f"streams={self.core.streams}: a residual of several streams and the hyper_connections arrangement go "
+                              f"together, in every layer")
+        if self.core.streams and self.depth_mix:
+            raise ConfigError("a depth mix over a residual of several streams is not built")
         for i, run in enumerate(self.schedule):
             if not 0 <= run.layer < len(self.layers):
                 raise ConfigError(f"schedule entry {i} names layer {run.layer} of {len(self.layers)}")

@@ -50,7 +50,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
                         const int* __restrict__ row_seg, const int* __restrict__ row_pos,
                         const int* __restrict__ block_tables, int table_stride, int heads, int kv_heads, int head_dim,
                         int page_size, int num_pages, int window, float scale_log2, int splits,
-                        float* __restrict__ part_o, float* __restrict__ part_ml, int keep_first, VecRef sink, int has_sink) {
+                        float* __restrict__ part_o, float* __restrict__ part_ml, int keep_first, VecRef sink, int has_sink, ScoreCap cap) {
     // `keep_first`: with a window, the request's first keys that stay visible; a row's visible keys are walked by an index
     // that counts them in ascending order (see jllm_kept_keys). `sink`: a number per query head whose exponential joins the
     // denominator (here where one block holds all of a row's keys, else in the combine kernel).
@@ -123,7 +123,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 const int key = key_at(base + tile * 8 + 2 * t + (i & 1));
-                s[tile][i] = key <= P ? s[tile][i] * scale_log2 : -INFINITY;
+                s[tile][i] = key <= P ? (cap ? cap(s[tile][i]) : s[tile][i] * scale_log2) : -INFINITY;
                 mx[i >> 1] = fmaxf(mx[i >> 1], s[tile][i]);
             }
         float corr[2];
@@ -314,10 +314,11 @@ int decode_split(const void* q, int q_stride, const void* k_cache, const void* v
                  const int* row_seg, const int* row_pos, const int* block_tables, int table_stride, int rows, int heads,
                  int kv_heads, int head_dim, int page_size, int window, float scale, int splits, float* scratch,
                  const staged::Fresh& fresh, cudaStream_t stream, int keep_first = 0, const void* sink = nullptr,
-                 int sink_dtype = JLLM_F32) {
+                 int sink_dtype = JLLM_F32, float softcap = 0.f) {
     // (kept first keys and a sink: the staged kernels of one block per (row, kv head, split) and the general kernel take them)
     const VecRef sk{sink, sink_dtype};
     const int has_sink = sink != nullptr;
+    const ScoreCap cap = score_cap(softcap, scale);
     JLLM_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention_decode: keep_first=%d needs a window", keep_first);
     JLLM_REQUIRE(rows >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && page_size > 0,
                  "attention_decode: rows=%d heads=%d kv_heads=%d page_size=%d", rows, heads, kv_heads, page_size);
@@ -346,7 +347,7 @@ int decode_split(const void* q, int q_stride, const void* k_cache, const void* v
 #define JLLM_STAGED(HD)                                                                                             \
     staged::launch<HD>(q, q_stride, k_cache, v_cache, out, out_stride, row_seg, row_pos, block_tables, table_stride, \
                        rows, heads, kv_heads, page_size, window, scale_log2, splits, part_o, part_ml, counters, fresh, stream, \
-                       keep_first, sk)
+                       keep_first, sk, cap)
         if (head_dim == 64) JLLM_STAGED(64); else if (head_dim == 128) JLLM_STAGED(128); else JLLM_STAGED(256);
 #undef JLLM_STAGED
         int rc2 = jllm_check_launch("attention_decode_staged");
@@ -364,7 +365,7 @@ int decode_split(const void* q, int q_stride, const void* k_cache, const void* v
                                                  (const __nv_bfloat16*)v_cache, (__nv_bfloat16*)out, out_stride,    \
                                                  row_seg, row_pos, block_tables, table_stride, heads, kv_heads,     \
                                                  head_dim, page_size, jllm_pool_pages(), window, scale_log2, splits, \
-                                                 part_o, part_ml, keep_first, sk, has_sink);                        \
+                                                 part_o, part_ml, keep_first, sk, has_sink, cap);                        \
     }
     if (hdc == 1) JLLM_LAUNCH(1) else if (hdc == 2) JLLM_LAUNCH(2) else if (hdc == 3) JLLM_LAUNCH(3) else JLLM_LAUNCH(4)
 #undef JLLM_LAUNCH
@@ -378,15 +379,15 @@ int decode_split(const void* q, int q_stride, const void* k_cache, const void* v
 }  // namespace
 
 // The same with a window that keeps the request's first `keep_first` keys visible and / or a sink per query head (`sink`
-// [heads] of type `sink_dtype`, or null).
+// [heads] of type `sink_dtype`, or null) and / or a cap on the scores (`softcap` > 0: s = softcap tanh(scale (q . k) / softcap)).
 JLLM_EXPORT int jllm_attention_decode_extras(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out,
                                              int out_stride, const int* row_seg, const int* row_pos, const int* block_tables,
                                              int table_stride, int rows, int heads, int kv_heads, int head_dim, int page_size,
                                              int window, float scale, int splits, float* scratch, int keep_first,
-                                             const void* sink, int sink_dtype, cudaStream_t stream) {
+                                             const void* sink, int sink_dtype, float softcap, cudaStream_t stream) {
     return decode_split(q, q_stride, k_cache, v_cache, out, out_stride, row_seg, row_pos, block_tables, table_stride, rows,
                         heads, kv_heads, head_dim, page_size, window, scale, splits, scratch, staged::Fresh{}, stream,
-                        keep_first, sink, sink_dtype);
+                        keep_first, sink, sink_dtype, softcap);
 }
 
 JLLM_EXPORT int jllm_attention_decode(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out,
@@ -409,7 +410,7 @@ namespace {
 int decode_flat(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out, int out_stride,
                 const int* row_seg, const int* row_pos, const int* block_tables, int table_stride, int rows, int heads,
                 int kv_heads, int head_dim, int page_size, int window, float scale, int blocks, float* scratch,
-                const staged::Fresh& fresh, cudaStream_t stream) {
+                const staged::Fresh& fresh, cudaStream_t stream, float softcap = 0.f) {
     JLLM_REQUIRE(rows >= 0 && rows <= staged::FLAT_MAX_ROWS && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 &&
                      page_size > 0 && heads / kv_heads <= 16,
                  "attention_decode_flat: rows=%d (at most %d) heads=%d kv_heads=%d page_size=%d", rows,
@@ -433,7 +434,8 @@ int decode_flat(const void* q, int q_stride, const void* k_cache, const void* v_
                             !g_separate_combine ? staged::pair_counters() : nullptr;
 #define JLLM_FLAT(HD)                                                                                                  \
     staged::launch_flat<HD>(q, q_stride, k_cache, v_cache, out, out_stride, row_seg, row_pos, block_tables, table_stride, \
-                            rows, heads, kv_heads, page_size, window, scale_log2, blocks, part_o, part_ml, counters, fresh, stream)
+                            rows, heads, kv_heads, page_size, window, scale_log2, blocks, part_o, part_ml, counters, fresh, stream, \
+                            score_cap(softcap, scale))
     if (head_dim == 64) JLLM_FLAT(64); else if (head_dim == 128) JLLM_FLAT(128); else JLLM_FLAT(256);
 #undef JLLM_FLAT
     return jllm_check_launch("attention_decode_flat");
@@ -444,9 +446,10 @@ int decode_flat(const void* q, int q_stride, const void* k_cache, const void* v_
 JLLM_EXPORT int jllm_attention_decode_flat(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out,
                                            int out_stride, const int* row_seg, const int* row_pos, const int* block_tables,
                                            int table_stride, int rows, int heads, int kv_heads, int head_dim, int page_size,
-                                           int window, float scale, int blocks, float* scratch, cudaStream_t stream) {
+                                           int window, float scale, int blocks, float* scratch, float softcap,
+                                           cudaStream_t stream) {
     return decode_flat(q, q_stride, k_cache, v_cache, out, out_stride, row_seg, row_pos, block_tables, table_stride, rows,
-                       heads, kv_heads, head_dim, page_size, window, scale, blocks, scratch, staged::Fresh{}, stream);
+                       heads, kv_heads, head_dim, page_size, window, scale, blocks, scratch, staged::Fresh{}, stream, softcap);
 }
 
 // Decode attention that first finishes its own row: `qkv` ([rows, stride]: query, key and value heads side by side) is as

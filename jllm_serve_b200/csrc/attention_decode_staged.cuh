@@ -93,6 +93,7 @@ struct Extras {
     int kept = 0;
     VecRef sink{nullptr, JLLM_F32};
     int has_sink = 0;
+    ScoreCap cap{0.f, 0.f};        // a cap on the scores
 };
 
 // The keys [first + tile_lo * 64, ...) of n_tiles tiles of one (row, kv head), for the G query heads of that kv head:
@@ -291,7 +292,7 @@ __device__ __forceinline__ void attend(uint8_t* smem_raw, const __nv_bfloat16* _
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int key = key0 + tile * 8 + 2 * t + (e & 1);
-                s[tile][e] = key <= P ? s[tile][e] * scale_log2 : -INFINITY;
+                s[tile][e] = key <= P ? (ex.cap ? ex.cap(s[tile][e]) : s[tile][e] * scale_log2) : -INFINITY;
                 mx[e >> 1] = fmaxf(mx[e >> 1], s[tile][e]);
             }
         float corr[2];
@@ -477,7 +478,8 @@ attention_decode_staged_kernel(const __nv_bfloat16* __restrict__ q, int q_stride
                                const int* __restrict__ row_pos, const int* __restrict__ block_tables, int table_stride,
                                int heads, int kv_heads, int page_size, int num_pages, int window, float scale_log2,
                                int splits, float* __restrict__ part_o, float* __restrict__ part_ml,
-                               int* __restrict__ counters, const Fresh fresh, int keep_first, VecRef sink, int has_sink) {
+                               int* __restrict__ counters, const Fresh fresh, int keep_first, VecRef sink, int has_sink,
+                               ScoreCap cap) {
     extern __shared__ __align__(128) uint8_t smem_raw[];
     const int r = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z;
     const int G = heads / kv_heads;
@@ -488,6 +490,7 @@ attention_decode_staged_kernel(const __nv_bfloat16* __restrict__ q, int q_stride
     ex.kept = jllm_kept_keys(jllm_first_key(P, window), window, keep_first);
     ex.sink = sink;
     ex.has_sink = has_sink;
+    ex.cap = cap;
     const int first = jllm_first_key(P, window) - ex.kept;      // the row's visible keys are numbered from here
     const int tiles_total = (P + 1 - first + TILE - 1) / TILE;
     const int tiles_per_split = (tiles_total + splits - 1) / splits;
@@ -544,7 +547,7 @@ attention_decode_flat_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, 
                              const int* __restrict__ row_seg, const int* __restrict__ row_pos,
                              const int* __restrict__ block_tables, int table_stride, int rows, int heads, int kv_heads,
                              int page_size, int num_pages, int window, float scale_log2, float* __restrict__ part_o,
-                             float* __restrict__ part_ml, int* __restrict__ counters, const Fresh fresh) {
+                             float* __restrict__ part_ml, int* __restrict__ counters, const Fresh fresh, ScoreCap cap) {
     extern __shared__ __align__(128) uint8_t smem_raw[];
     __shared__ int s_cum[FLAT_MAX_ROWS + 1];
     pdl_wait();
@@ -552,6 +555,8 @@ attention_decode_flat_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, 
     if (threadIdx.x < 32) flat_prefix(row_pos, rows, window, s_cum);
     __syncthreads();
     const int G = heads / kv_heads;
+    Extras ex;
+    ex.cap = cap;
     const long long all = (long long)kv_heads * s_cum[rows];
     long long at = all * blockIdx.x / gridDim.x;
     const long long end = all * (blockIdx.x + 1) / gridDim.x;
@@ -577,7 +582,7 @@ attention_decode_flat_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, 
         attend<HD>(smem_raw, q, q_stride, k_cache, v_cache, out, out_stride, block_tables + (size_t)row_seg[r] * table_stride,
                    table_stride, num_pages, heads, kv_heads, page_size, scale_log2, r, kvh, P, first, tile_lo, n, alone,
                    part_o + slot * G * HD,
-                   (size_t)HD, part_ml + slot * G * 2, (size_t)2, fresh);
+                   (size_t)HD, part_ml + slot * G * 2, (size_t)2, fresh, false, ex);
         at += n;
         if (counters != nullptr && !alone && last_of_pair(counters + (size_t)r * kv_heads + kvh, parts)) {
             const size_t slot0 = (size_t)r * kv_heads + kvh + b_first;      // the slots of the pair's parts follow one another
@@ -647,7 +652,7 @@ template <int HD>
 void launch_flat(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out, int out_stride,
                  const int* row_seg, const int* row_pos, const int* block_tables, int table_stride, int rows, int heads,
                  int kv_heads, int page_size, int window, float scale_log2, int blocks, float* part_o, float* part_ml,
-                 int* counters, const Fresh& fresh, cudaStream_t stream) {
+                 int* counters, const Fresh& fresh, cudaStream_t stream, ScoreCap cap) {
     const size_t stage_bytes = (size_t)STAGES * 2 * TILE * HD * 2;
     const size_t merge_bytes = ((size_t)WARPS * 16 * HD + WARPS * 16 * 2) * sizeof(float);
     const size_t smem = 16 * HD * 2 + (stage_bytes > merge_bytes ? stage_bytes : merge_bytes);
@@ -656,7 +661,7 @@ void launch_flat(const void* q, int q_stride, const void* k_cache, const void* v
     jllm_launch(kern, dim3(blocks), dim3(THREADS), smem, stream, true, (const __nv_bfloat16*)q, q_stride,
                 (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, (__nv_bfloat16*)out, out_stride, row_seg,
                 row_pos, block_tables, table_stride, rows, heads, kv_heads, page_size, jllm_pool_pages(), window, scale_log2,
-                part_o, part_ml, counters, fresh);
+                part_o, part_ml, counters, fresh, cap);
     if (counters == nullptr)
         jllm_launch(attention_combine_flat_kernel, dim3(rows, heads), dim3(128), 0, stream, true, (const float*)part_o,
                     (const float*)part_ml, (__nv_bfloat16*)out, out_stride, row_pos, rows, heads, kv_heads, HD, window,
@@ -667,7 +672,7 @@ template <int HD>
 void launch(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out, int out_stride,
             const int* row_seg, const int* row_pos, const int* block_tables, int table_stride, int rows, int heads,
             int kv_heads, int page_size, int window, float scale_log2, int splits, float* part_o, float* part_ml,
-            int* counters, const Fresh& fresh, cudaStream_t stream, int keep_first = 0, VecRef sink = VecRef{nullptr, JLLM_F32}) {
+            int* counters, const Fresh& fresh, cudaStream_t stream, int keep_first, VecRef sink, ScoreCap cap) {
     const size_t stage_bytes = (size_t)STAGES * 2 * TILE * HD * 2;
     const size_t merge_bytes = ((size_t)WARPS * 16 * HD + WARPS * 16 * 2) * sizeof(float);
     const size_t smem = 16 * HD * 2 + (stage_bytes > merge_bytes ? stage_bytes : merge_bytes);
@@ -677,7 +682,7 @@ void launch(const void* q, int q_stride, const void* k_cache, const void* v_cach
         (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache,
         (__nv_bfloat16*)out, out_stride, row_seg, row_pos, block_tables, table_stride, heads, kv_heads, page_size,
         jllm_pool_pages(), window, scale_log2, splits, part_o, part_ml, counters, fresh, keep_first, sink,
-        (int)(sink.p != nullptr));
+        (int)(sink.p != nullptr), cap);
 }
 
 // The library's pair counters on the current device (nullptr: the combine kernels run instead).

@@ -5,7 +5,8 @@
 //                    once with a gain per column; rotation of the first rotary_dim values of every map; then
 //                      * query (head h, map m) to its own row of `width` values, its `dim` values at place m * dim, zeros elsewhere;
 //                      * the maps of a key head side by side into ONE cached row of `width` values, zeros behind them;
-//                      * the value into the value row, zeros behind it.
+//                      * the value into the value row, zeros behind it (v_off = k_off: the values are the keys as projected).
+//                    Queries may grow with their position: q times 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).
 //                    A query's dot product with a cached row is then the dot product with its own map alone, so an attention with
 //                    heads x maps query heads and kv_heads key / value heads of one width computes all maps over values that are
 //                    cached once, on the kernels that were built for plain heads.
@@ -45,6 +46,8 @@ __device__ __forceinline__ void store_piece(T* p, const float (&o)[N]) {
 struct MapShape {
     int heads, kv_heads, maps, dim, vdim, width, page_size, rotary_dim, pairing;
     int ld, k_off, v_off, ld_q;
+    int temp_every;            // 0: the queries are not multiplied
+    float temp_coef;
 };
 
 // One block per row. N values a thread at a time (N > 1 only where every piece of every part is whole and aligned).
@@ -114,10 +117,17 @@ map_prepare_kernel(const T* __restrict__ src, MapShape s, const float* __restric
         }
     };
     const int W = s.width;
+    const float temp = s.temp_every > 0 ? fmaf(s.temp_coef, logf((float)((positions[r] + 1) / s.temp_every + 1)), 1.f) : 1.f;
     for (int e = tid * N; e < s.heads * s.maps * W; e += blockDim.x * N) {
         const int hm = e / W, i = e - hm * W - (hm % s.maps) * s.dim;
         float o[N] = {};
-        if (i >= 0 && i < s.dim) take(row, q_gain, inv_q, hm * s.dim, i, o);
+        if (i >= 0 && i < s.dim) {
+            take(row, q_gain, inv_q, hm * s.dim, i, o);
+            if (s.temp_every > 0) {
+#pragma unroll
+                for (int k = 0; k < N; ++k) o[k] = __fmul_rn(o[k], temp);
+            }
+        }
         store_piece<T, N>(q_out + r * s.ld_q + e, o);
     }
     if (!write_kv) return;
@@ -200,14 +210,14 @@ JLLM_EXPORT int jllm_map_prepare(const void* src, int dtype, int ld, int k_off, 
                                  float eps, const float* cos_t, const float* sin_t, int rotary_dim, int pairing, const int* positions,
                                  const int* slots, void* q_out, int ld_q, void* k_cache, void* v_cache, int write_kv, int rows,
                                  int heads, int kv_heads, int maps, int dim, int vdim, int width, int page_size,
-                                 cudaStream_t stream) {
+                                 int temp_every, float temp_coef, cudaStream_t stream) {
     JLLM_REQUIRE(rows >= 0 && heads > 0 && kv_heads > 0 && maps > 0 && dim > 0 && vdim > 0, "map_prepare: rows=%d heads=%d/%d maps=%d dim=%d/%d",
                  rows, heads, kv_heads, maps, dim, vdim);
     JLLM_REQUIRE(width >= maps * dim && width >= vdim && ld_q >= heads * maps * width, "map_prepare: width=%d for %d maps of %d and values of %d",
                  width, maps, dim, vdim);
     JLLM_REQUIRE(rotary_dim >= 0 && rotary_dim <= dim && rotary_dim % 2 == 0, "map_prepare: rotary_dim=%d dim=%d", rotary_dim, dim);
     if (rows == 0) return JLLM_OK;
-    const MapShape s{heads, kv_heads, maps, dim, vdim, width, page_size, rotary_dim, pairing, ld, k_off, v_off, ld_q};
+    const MapShape s{heads, kv_heads, maps, dim, vdim, width, page_size, rotary_dim, pairing, ld, k_off, v_off, ld_q, temp_every, temp_coef};
     const int num_slots = jllm_pool_pages() * page_size;
     const int per = dtype == JLLM_F32 ? 4 : 8;
     auto whole = [&](long long n) { return n % per == 0; };

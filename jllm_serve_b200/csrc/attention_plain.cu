@@ -11,7 +11,8 @@
 // Two things a mixer may add. `keep_first` > 0 (with a window): the request's first keep_first keys stay visible to every
 // later row, so a row sees [0, keep_first) and [first, P]; the keys in between are passed over. `sink` (one number per query
 // head, else null): the softmax's denominator also holds exp(sink[h]), a key without a value that is not multiplied by the
-// scale; the running maximum starts from it, so nothing overflows whichever is larger.
+// scale; the running maximum starts from it, so nothing overflows whichever is larger. And a cap on the scores (`softcap` > 0):
+// s = softcap * tanh(scale (q . k) / softcap).
 //
 // Layouts: q [rows, q_stride] with head h at h * head_dim; cache K and V
 // [pages, kv_heads, page_size, cache_dim], a key in the first head_dim values of its row and a value in the first
@@ -31,7 +32,7 @@ attention_plain_kernel(const T* __restrict__ q, int q_stride, const T* __restric
                        const int* __restrict__ row_seg, const int* __restrict__ row_pos,
                        const int* __restrict__ block_tables, int table_stride, int heads, int kv_heads, int head_dim,
                        int value_dim, int cache_dim, int page_size, int num_pages, int window, float scale, int keep_first,
-                       VecRef sink, int has_sink) {
+                       VecRef sink, int has_sink, float softcap) {
     extern __shared__ float smem[];
     float* qs = smem;                  // head_dim
     float* es = qs + head_dim;         // THREADS
@@ -56,7 +57,8 @@ attention_plain_kernel(const T* __restrict__ q, int q_stride, const T* __restric
         if (kCheckBounds && kr == nullptr) return -INFINITY;
         float acc = 0.f;
         for (int i = 0; i < head_dim; ++i) acc = fmaf(qs[i], to_float(kr[i]), acc);
-        return __fmul_rn(acc, scale);
+        const float scaled = __fmul_rn(acc, scale);
+        return softcap > 0.f ? __fmul_rn(softcap, tanhf(scaled / softcap)) : scaled;
     };
 
     // the visible keys in ascending order: index u < kept is key u, index u >= kept is key first + (u - kept)
@@ -103,7 +105,7 @@ JLLM_EXPORT int jllm_attention_plain(const void* q, int q_stride, const void* k_
                                      int out_stride, const int* row_seg, const int* row_pos, const int* block_tables,
                                      int table_stride, int rows, int heads, int kv_heads, int head_dim, int value_dim,
                                      int cache_dim, int page_size, int window, float scale, int dtype, int keep_first,
-                                     const void* sink, int sink_dtype, cudaStream_t stream) {
+                                     const void* sink, int sink_dtype, float softcap, cudaStream_t stream) {
     JLLM_REQUIRE(rows >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && head_dim > 0 && page_size > 0,
                  "attention: rows=%d heads=%d kv_heads=%d head_dim=%d page_size=%d", rows, heads, kv_heads, head_dim,
                  page_size);
@@ -124,11 +126,11 @@ JLLM_EXPORT int jllm_attention_plain(const void* q, int q_stride, const void* k_
         attention_plain_kernel<float><<<grid, THREADS, smem, stream>>>(
             (const float*)q, q_stride, (const float*)k_cache, (const float*)v_cache, (float*)out, out_stride, row_seg,
             row_pos, block_tables, table_stride, heads, kv_heads, head_dim, value_dim, cache_dim, page_size, num_pages, window, scale,
-            keep_first, sk, has_sink);
+            keep_first, sk, has_sink, softcap);
     else
         attention_plain_kernel<__nv_bfloat16><<<grid, THREADS, smem, stream>>>(
             (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache,
             (__nv_bfloat16*)out, out_stride, row_seg, row_pos, block_tables, table_stride, heads, kv_heads, head_dim,
-            value_dim, cache_dim, page_size, num_pages, window, scale, keep_first, sk, has_sink);
+            value_dim, cache_dim, page_size, num_pages, window, scale, keep_first, sk, has_sink, softcap);
     return jllm_check_launch("attention_plain");
 }

@@ -62,7 +62,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
                          const int* __restrict__ seg_start, const int* __restrict__ seg_len,
                          const int* __restrict__ seg_kv_len, const int* __restrict__ block_tables, int table_stride,
                          int num_segs, int heads, int kv_heads, int page_size, int num_pages, int window,
-                         float scale_log2, int keep_first, VecRef sink, int has_sink) {
+                         float scale_log2, int keep_first, VecRef sink, int has_sink, ScoreCap cap) {
     // `keep_first`: with a window, the request's first keys that stay visible to every row: the key tiles that hold them are
     // walked in front of the window's tiles. `sink`: a number per query head whose exponential joins the denominator.
     constexpr int CHUNKS = HD / 8;               // 16-byte chunks per row
@@ -179,7 +179,14 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
                     mma_16816(s[2 * jp + 1], qf[ks], kf[2], kf[3]);
                 }
             }
-            // ---- mask and online softmax ----
+            // ---- cap, mask and online softmax ----
+            const float to_log2 = cap ? 1.f : scale_log2;      // (a capped score is in base 2 already)
+            if (cap) {
+    #pragma unroll
+                for (int j = 0; j < BKV / 8; ++j)
+    #pragma unroll
+                    for (int i = 0; i < 4; ++i) s[j][i] = cap(s[j][i]);
+            }
             const int key0 = kt * BKV;
             float mx[2] = {-INFINITY, -INFINITY};
             // a tile that every row of this warp sees whole (all keys at or before the warp's first position and
@@ -191,7 +198,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
                 for (int j = 0; j < BKV / 8; ++j)
     #pragma unroll
                     for (int i = 0; i < 4; ++i) {
-                        s[j][i] *= scale_log2;
+                        s[j][i] *= to_log2;
                         mx[i >> 1] = fmaxf(mx[i >> 1], s[j][i]);
                     }
             } else {
@@ -201,7 +208,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
                     for (int i = 0; i < 4; ++i) {
                         const int key = key0 + j * 8 + 2 * t + (i & 1), P = pos_r[i >> 1];
                         const bool vis = jllm_key_visible(key, P, first_r[i >> 1], keep);
-                        s[j][i] = vis ? s[j][i] * scale_log2 : -INFINITY;
+                        s[j][i] = vis ? s[j][i] * to_log2 : -INFINITY;
                         mx[i >> 1] = fmaxf(mx[i >> 1], s[j][i]);
                     }
             }
@@ -275,7 +282,7 @@ template <int HD>
 int launch(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out, int out_stride,
            const int* seg_start, const int* seg_len, const int* seg_kv_len, const int* block_tables, int table_stride,
            int num_segs, int rows, int heads, int kv_heads, int page_size, int window, float scale,
-           cudaStream_t stream, int keep_first = 0, VecRef sink = VecRef{nullptr, JLLM_F32}) {
+           cudaStream_t stream, int keep_first, VecRef sink, float softcap) {
     const size_t smem = (size_t)BQ * HD * 2 + 4 * (size_t)BKV * HD * 2;
     auto kern = attention_prefill_kernel<HD>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -284,7 +291,7 @@ int launch(const void* q, int q_stride, const void* k_cache, const void* v_cache
                                           (const __nv_bfloat16*)v_cache, (__nv_bfloat16*)out, out_stride, seg_start,
                                           seg_len, seg_kv_len, block_tables, table_stride, num_segs, heads, kv_heads,
                                           page_size, jllm_pool_pages(), window, scale * LOG2E, keep_first, sink,
-                                          (int)(sink.p != nullptr));
+                                          (int)(sink.p != nullptr), score_cap(softcap, scale));
     return jllm_check_launch("attention_prefill");
 }
 
@@ -298,7 +305,7 @@ static int prefill_any(const void* q, int q_stride, const void* k_cache, const v
                                        int out_stride, const int* seg_start, const int* seg_len, const int* seg_kv_len,
                                        const int* block_tables, int table_stride, int num_segs, int rows, int heads,
                                        int kv_heads, int head_dim, int page_size, int window, float scale,
-                                       cudaStream_t stream, int keep_first, VecRef sink) {
+                                       cudaStream_t stream, int keep_first, VecRef sink, float softcap) {
     JLLM_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention_prefill: keep_first=%d needs a window", keep_first);
     JLLM_REQUIRE(rows >= 0 && num_segs >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && page_size > 0,
                  "attention_prefill: rows=%d segments=%d heads=%d kv_heads=%d page_size=%d", rows, num_segs, heads,
@@ -310,7 +317,7 @@ static int prefill_any(const void* q, int q_stride, const void* k_cache, const v
     JLLM_REQUIRE(heads <= 65535, "attention_prefill: heads=%d", heads);
     if (rows == 0 || num_segs == 0) return JLLM_OK;
 #define JLLM_ARGS q, q_stride, k_cache, v_cache, out, out_stride, seg_start, seg_len, seg_kv_len, block_tables, \
-                  table_stride, num_segs, rows, heads, kv_heads, page_size, window, scale, stream, keep_first, sink
+                  table_stride, num_segs, rows, heads, kv_heads, page_size, window, scale, stream, keep_first, sink, softcap
     if (head_dim == 64) return launch<64>(JLLM_ARGS);
     if (head_dim == 128) return launch<128>(JLLM_ARGS);
     return launch<256>(JLLM_ARGS);
@@ -323,16 +330,18 @@ JLLM_EXPORT int jllm_attention_prefill(const void* q, int q_stride, const void* 
                                        int kv_heads, int head_dim, int page_size, int window, float scale,
                                        cudaStream_t stream) {
     return prefill_any(q, q_stride, k_cache, v_cache, out, out_stride, seg_start, seg_len, seg_kv_len, block_tables, table_stride,
-                       num_segs, rows, heads, kv_heads, head_dim, page_size, window, scale, stream, 0, VecRef{nullptr, JLLM_F32});
+                       num_segs, rows, heads, kv_heads, head_dim, page_size, window, scale, stream, 0, VecRef{nullptr, JLLM_F32}, 0.f);
 }
 
-// The same with a window that keeps the request's first `keep_first` keys visible and / or a sink per query head.
+// The same with a window that keeps the request's first `keep_first` keys visible and / or a sink per query head and / or a cap on the
+// scores (`softcap` > 0: s = softcap tanh(scale (q . k) / softcap)).
 JLLM_EXPORT int jllm_attention_prefill_extras(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out,
                                               int out_stride, const int* seg_start, const int* seg_len, const int* seg_kv_len,
                                               const int* block_tables, int table_stride, int num_segs, int rows, int heads,
                                               int kv_heads, int head_dim, int page_size, int window, float scale,
-                                              int keep_first, const void* sink, int sink_dtype, cudaStream_t stream) {
+                                              int keep_first, const void* sink, int sink_dtype, float softcap,
+                                              cudaStream_t stream) {
     return prefill_any(q, q_stride, k_cache, v_cache, out, out_stride, seg_start, seg_len, seg_kv_len, block_tables, table_stride,
                        num_segs, rows, heads, kv_heads, head_dim, page_size, window, scale, stream, keep_first,
-                       VecRef{sink, sink_dtype});
+                       VecRef{sink, sink_dtype}, softcap);
 }

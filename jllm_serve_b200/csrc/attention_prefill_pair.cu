@@ -16,6 +16,8 @@
 // grew by more than 2^8 (the reference point of the exponentials stays until then).
 // Every mbarrier wait is bounded; a wait that runs out raises the error word and all roles leave.
 //
+// A cap on the scores (`softcap` > 0: s = softcap tanh(scale (q . k) / softcap)) is applied to a row of S as it leaves tensor memory.
+//
 // Requirements: bfloat16, head_dim 128, page_size a power of two <= 128, 16-byte aligned q rows.
 #include "tcgen05_common.cuh"
 
@@ -48,7 +50,7 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
                               const int* __restrict__ seg_start, const int* __restrict__ seg_len,
                               const int* __restrict__ seg_kv_len, const int* __restrict__ block_tables,
                               int table_stride, int num_segs, int heads, int kv_heads, int page_size, int page_shift,
-                              int num_pages, int window, float scale_log2, int* __restrict__ error_word) {
+                              int num_pages, int window, float scale_log2, int* __restrict__ error_word, ScoreCap cap) {
     extern __shared__ uint8_t smem_raw[];
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
     uint8_t* aligned = smem_raw + (base - smem_u32(smem_raw));
@@ -227,6 +229,7 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
             const int P = pos0 + x * BQ + min(r, rows_x[x] - 1);   // rows past the end copy the last row, and are not stored
             const int lo = jllm_first_key(P, window);              // the first key this row sees (window or chunk)
             const int pos0_x = pos0 + x * BQ;
+            const float to_log2 = cap ? 1.f : scale_log2;          // (a capped score is in base 2 already)
             float m = -INFINITY, l = 0.f;
             bool ok = true;
             for (int j = 0; j < n_mine && ok; ++j) {
@@ -238,6 +241,12 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
 #pragma unroll
                 for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, v[c]);
                 tmem_ld_wait();
+                if (cap) {
+#pragma unroll
+                    for (int c = 0; c < 4; ++c)
+#pragma unroll
+                        for (int i = 0; i < 32; ++i) v[c][i] = __float_as_uint(cap(__uint_as_float(v[c][i])));
+                }
                 if (masked) {
 #pragma unroll
                     for (int c = 0; c < 4; ++c)
@@ -255,7 +264,7 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
 #pragma unroll
                     for (int i = 0; i < 32; ++i) mxs[i & 3] = fmaxf(mxs[i & 3], __uint_as_float(v[c][i]));
                 const float mx = fmaxf(fmaxf(mxs[0], mxs[1]), fmaxf(mxs[2], mxs[3]));
-                const float m_cand = fmaxf(m, mx * scale_log2);
+                const float m_cand = fmaxf(m, mx * to_log2);
                 const float m_new = (m_cand - m > 8.f) ? m_cand : m;
                 const float m_use = m_new == -INFINITY ? 0.f : m_new;
                 const float corr = fast_exp2(m - m_use);
@@ -268,8 +277,8 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
                     for (int c = 0; c < 2; ++c)
 #pragma unroll
                         for (int i = 0; i < 32; i += 2) {
-                            const float p0 = fast_exp2(fmaf(__uint_as_float(v[2 * half + c][i]), scale_log2, -m_use));
-                            const float p1 = fast_exp2(fmaf(__uint_as_float(v[2 * half + c][i + 1]), scale_log2, -m_use));
+                            const float p0 = fast_exp2(fmaf(__uint_as_float(v[2 * half + c][i]), to_log2, -m_use));
+                            const float p1 = fast_exp2(fmaf(__uint_as_float(v[2 * half + c][i + 1]), to_log2, -m_use));
                             sums[(i >> 1) & 1] += p0 + p1;
                             __nv_bfloat162 b2 = __floats2bfloat162_rn(p0, p1);
                             pk[(c * 32 + i) >> 1] = *reinterpret_cast<uint32_t*>(&b2);
@@ -340,7 +349,8 @@ JLLM_EXPORT int jllm_attention_prefill_pair(const void* q, int q_stride, const v
                                             long long cache_pages, void* out, int out_stride, const int* seg_start,
                                             const int* seg_len, const int* seg_kv_len, const int* block_tables,
                                             int table_stride, int num_segs, int rows, int heads, int kv_heads,
-                                            int head_dim, int page_size, int window, float scale, cudaStream_t stream) {
+                                            int head_dim, int page_size, int window, float scale, float softcap,
+                                            cudaStream_t stream) {
     JLLM_REQUIRE(rows >= 0 && num_segs >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && cache_pages > 0,
                  "attention_prefill_pair: rows=%d segments=%d heads=%d kv_heads=%d pages=%lld", rows, num_segs, heads,
                  kv_heads, cache_pages);
@@ -372,6 +382,6 @@ JLLM_EXPORT int jllm_attention_prefill_pair(const void* q, int q_stride, const v
     jllm_launch(kern, grid, dim3(THREADS), SMEM_BYTES, stream, true, map_q, map_k, map_v, (const __nv_bfloat16*)k_cache,
                 (const __nv_bfloat16*)v_cache, (__nv_bfloat16*)out, out_stride, seg_start, seg_len, seg_kv_len,
                 block_tables, table_stride, num_segs, heads, kv_heads, page_size, page_shift, (int)cache_pages, window,
-                scale * LOG2E, error_word);
+                scale * LOG2E, error_word, score_cap(softcap, scale));
     return jllm_check_launch("attention_prefill_pair");
 }

@@ -40,7 +40,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ seg_start, const int* __restrict__ seg_len,
                             const int* __restrict__ seg_kv_len, const int* __restrict__ block_tables, int table_stride,
                             int num_segs, int heads, int kv_heads, int page_size, int page_shift, int num_pages, int window,
-                            float scale_log2, int* __restrict__ error_word, int keep_first, VecRef sink, int has_sink) {
+                            float scale_log2, int* __restrict__ error_word, int keep_first, VecRef sink, int has_sink, ScoreCap cap) {
     // `keep_first`: with a window, the request's first keys that stay visible to every row: the key tiles that hold them are
     // walked in front of the window's tiles (tile j of the walk is key tile tile_of(j)). `sink`: a number per query head
     // whose exponential joins the row's sum at the end.
@@ -212,6 +212,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const uint32_t lane_addr = tmem_base + ((uint32_t)(quad * 32) << 16);
         const int P = pos0 + min(r, rows_here - 1);            // rows past the end copy the last row, and are not stored
         const int lo = jllm_first_key(P, window);              // the first key this row sees (window or chunk)
+        const float to_log2 = cap ? 1.f : scale_log2;          // (a capped score is in base 2 already)
         float m = -INFINITY, l = 0.f;
         bool ok = true;
         for (int j = 0; j < n_tiles && ok; ++j) {
@@ -225,6 +226,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
             for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(lane_addr + b * 128 + c * 32, v[c]);
             tmem_ld_wait();
+            if (cap) {
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) v[c][i] = __float_as_uint(cap(__uint_as_float(v[c][i])));
+            }
             if (masked) {
 #pragma unroll
                 for (int c = 0; c < 4; ++c)
@@ -243,7 +250,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             const float mx = fmaxf(fmaxf(mxs[0], mxs[1]), fmaxf(mxs[2], mxs[3]));
             // The reference point of the exponentials only moves when the maximum grew by more than 2^8: until
             // then p stays below 256, which bfloat16 and the float32 sum hold as well, and O needs no rescaling.
-            const float m_cand = fmaxf(m, mx * scale_log2);
+            const float m_cand = fmaxf(m, mx * to_log2);
             const float m_new = (m_cand - m > 8.f) ? m_cand : m;
             const float m_use = m_new == -INFINITY ? 0.f : m_new;
             const float corr = fast_exp2(m - m_use);
@@ -254,8 +261,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             for (int c = 0; c < 4; ++c)
 #pragma unroll
                 for (int i = 0; i < 32; i += 2) {
-                    const float p0 = fast_exp2(fmaf(__uint_as_float(v[c][i]), scale_log2, -m_use));
-                    const float p1 = fast_exp2(fmaf(__uint_as_float(v[c][i + 1]), scale_log2, -m_use));
+                    const float p0 = fast_exp2(fmaf(__uint_as_float(v[c][i]), to_log2, -m_use));
+                    const float p1 = fast_exp2(fmaf(__uint_as_float(v[c][i + 1]), to_log2, -m_use));
                     sum += p0 + p1;
                     __nv_bfloat162 b2 = __floats2bfloat162_rn(p0, p1);
                     pk[(c * 32 + i) >> 1] = *reinterpret_cast<uint32_t*>(&b2);
@@ -367,7 +374,7 @@ static int prefill_tc_any(const void* q, int q_stride, const void* k_cache, cons
                                           const int* seg_len, const int* seg_kv_len, const int* block_tables,
                                           int table_stride, int num_segs, int rows, int heads, int kv_heads,
                                           int head_dim, int page_size, int window, float scale, cudaStream_t stream,
-                                          int keep_first, VecRef sink) {
+                                          int keep_first, VecRef sink, float softcap) {
     JLLM_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention_prefill_tc: keep_first=%d needs a window", keep_first);
     JLLM_REQUIRE(rows >= 0 && num_segs >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && cache_pages > 0,
                  "attention_prefill_tc: rows=%d segments=%d heads=%d kv_heads=%d pages=%lld", rows, num_segs, heads,
@@ -397,7 +404,7 @@ static int prefill_tc_any(const void* q, int q_stride, const void* k_cache, cons
     jllm_launch(kern, grid, dim3(THREADS), SMEM_BYTES, stream, true, map_q, map_k, map_v, (const __nv_bfloat16*)k_cache,
                 (const __nv_bfloat16*)v_cache, (__nv_bfloat16*)out, out_stride, seg_start, seg_len, seg_kv_len,
                 block_tables, table_stride, num_segs, heads, kv_heads, page_size, page_shift, (int)cache_pages, window,
-                scale * LOG2E, error_word, keep_first, sink, (int)(sink.p != nullptr));
+                scale * LOG2E, error_word, keep_first, sink, (int)(sink.p != nullptr), score_cap(softcap, scale));
     return jllm_check_launch("attention_prefill_tc");
 }
 
@@ -408,17 +415,18 @@ JLLM_EXPORT int jllm_attention_prefill_tc(const void* q, int q_stride, const voi
                                           int head_dim, int page_size, int window, float scale, cudaStream_t stream) {
     return prefill_tc_any(q, q_stride, k_cache, v_cache, cache_pages, out, out_stride, seg_start, seg_len, seg_kv_len, block_tables,
                           table_stride, num_segs, rows, heads, kv_heads, head_dim, page_size, window, scale, stream, 0,
-                          VecRef{nullptr, JLLM_F32});
+                          VecRef{nullptr, JLLM_F32}, 0.f);
 }
 
-// The same with a window that keeps the request's first `keep_first` keys visible and / or a sink per query head.
+// The same with a window that keeps the request's first `keep_first` keys visible and / or a sink per query head and / or a cap on
+// the scores (`softcap` > 0: s = softcap tanh(scale (q . k) / softcap)).
 JLLM_EXPORT int jllm_attention_prefill_tc_extras(const void* q, int q_stride, const void* k_cache, const void* v_cache,
                                                  long long cache_pages, void* out, int out_stride, const int* seg_start,
                                                  const int* seg_len, const int* seg_kv_len, const int* block_tables,
                                                  int table_stride, int num_segs, int rows, int heads, int kv_heads,
                                                  int head_dim, int page_size, int window, float scale, int keep_first,
-                                                 const void* sink, int sink_dtype, cudaStream_t stream) {
+                                                 const void* sink, int sink_dtype, float softcap, cudaStream_t stream) {
     return prefill_tc_any(q, q_stride, k_cache, v_cache, cache_pages, out, out_stride, seg_start, seg_len, seg_kv_len, block_tables,
                           table_stride, num_segs, rows, heads, kv_heads, head_dim, page_size, window, scale, stream, keep_first,
-                          VecRef{sink, sink_dtype});
+                          VecRef{sink, sink_dtype}, softcap);
 }

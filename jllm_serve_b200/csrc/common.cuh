@@ -191,6 +191,54 @@ __device__ __forceinline__ float glu_unit(float gate, float up, int word) {
     return __fmul_rn(glu_act<FAST>(gate, word), up);
 }
 
+// What a product's epilogue is told about the gated unit it applies: `word` as above (0: no gating). A mixture of experts whose
+// units are stacked in one product says more: units from `split` on are another feed-forward's (a shared expert's) with a word of
+// their own, and with `weights` ([rows, ld_w] float32) unit u's result is multiplied by weights[row, u / ff], a unit's from `split`
+// on by weights[row, split / ff].
+struct GluArgs {
+    int word, word_behind, split, ff, ld_w;
+    const float* weights;
+    __host__ __device__ __forceinline__ explicit operator bool() const { return word != 0; }
+    __device__ __forceinline__ int word_of(int unit) const { return unit < split ? word : word_behind; }
+    __device__ __forceinline__ float weight(int row, int unit) const {
+        return weights[(size_t)row * ld_w + min((unit < split ? unit : split) / ff, ld_w - 1)];
+    }
+    // whether eight units from a multiple of 8 on always share their word and their weight
+    __device__ __forceinline__ bool in_eights() const { return (ff & 7) == 0 && ((split & 7) == 0 || split == 0x7fffffff); }
+    template <bool FAST>
+    __device__ __forceinline__ float apply(float gate, float up, int row, int unit) const {
+        const float y = glu_unit<FAST>(gate, up, word_of(unit));
+        return weights != nullptr ? __fmul_rn(y, weight(row, unit)) : y;
+    }
+};
+// ... from a launcher's two arguments: the word, and (or null) a host struct of what is said beyond it
+struct GluMore {
+    int word_behind, split, ff, ld_w;
+    const float* weights;
+};
+inline GluArgs glu_args(int word, const void* more) {
+    if (more == nullptr) return GluArgs{word, word, 0x7fffffff, 1, 0, nullptr};
+    const GluMore& m = *static_cast<const GluMore*>(more);
+    return GluArgs{word, m.split > 0 ? m.word_behind : word, m.split > 0 ? m.split : 0x7fffffff, m.ff > 0 ? m.ff : 1, m.ld_w, m.weights};
+}
+
+// ---- scores under a cap: c tanh(s / c) ------------------------------------------------------------------------
+// tanh(x) = 1 - 2 / (e^(2x) + 1) by the special-function unit's exponential and reciprocal: within a few units of the seventh
+// digit of 1 everywhere (an error in the SCORE of that times the cap), and exactly +-1 far out.
+__device__ __forceinline__ float unit_tanh(float x) {
+    float t;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(t) : "f"(x * 2.885390081777927f));      // 2 log2(e)
+    return 1.f - __fdividef(2.f, t + 1.f);
+}
+// What the bfloat16 attention kernels are told: a raw dot product d becomes the base-2 score out * tanh(in * d) with in =
+// scale / cap and out = cap * log2(e). out = 0: no cap.
+struct ScoreCap {
+    float in, out;
+    __host__ __device__ __forceinline__ explicit operator bool() const { return out != 0.f; }
+    __device__ __forceinline__ float operator()(float d) const { return out * unit_tanh(in * d); }
+};
+inline ScoreCap score_cap(float cap, float scale) { return cap > 0.f ? ScoreCap{scale / cap, cap * 1.4426950408889634f} : ScoreCap{0.f, 0.f}; }
+
 // What a product does with its result, the launchers' `accumulate` argument: 0 store it, 1 add it to what `out` holds, 2
 // store max(v, 0)^2 (the activation of an ungated feed-forward; behind the bias).
 enum : int { EPI_STORE = 0, EPI_ADD = 1, EPI_RELU2 = 2 };

@@ -10,7 +10,7 @@
 // What a design may ask of the router beyond that: scores that are a softmax over all entries instead of a logistic function
 // of each (`softmax`); entries behind the experts that have no weights and hand the row through as it is (`identity`: the
 // router matrix has experts + identity rows, the chosen identity entries' weights leave as ONE number, their sum, in the
-// column behind the experts' and the gates'); and rows behind those that are not routed at all but give a logistic gate per
+// column behind the experts' and the gates'); a bias on the entries' logits, in front of the scores (`bias`); and rows behind those that are not routed at all but give a logistic gate per
 // row (`gates`: a shared expert's), which leave in the columns behind the experts'.
 #include "common.cuh"
 
@@ -18,7 +18,7 @@ namespace {
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-route_experts_kernel(const T* __restrict__ h, int ld, const float* __restrict__ router, VecRef correction, int has_correction,
+route_experts_kernel(const T* __restrict__ h, int ld, const float* __restrict__ router, VecRef bias, int has_bias, VecRef correction, int has_correction,
                      float* __restrict__ weights, int dim, int real, int top, float scale, int normalize, int identity, int gates,
                      int softmax, int ld_out) {
     // `real` experts have weights; entries [real, real + identity) hand the row through; rows [entries, entries + gates) of the
@@ -63,6 +63,7 @@ route_experts_kernel(const T* __restrict__ h, int ld, const float* __restrict__ 
         }
         acc = warp_sum(acc);
         if (lane == 0) {
+            if (has_bias && e < entries) acc += bias[e];
             const float sc = (softmax && e < entries) ? acc : 1.f / (1.f + expf(-acc));
             s[e] = sc;
             c[e] = (has_correction && e < entries) ? sc + correction[e] : sc;
@@ -146,25 +147,34 @@ __global__ void scale_expert_hidden_vec_kernel(T* __restrict__ hidden, const flo
 // 2 * width]: all gate values, then all up values; width = experts * ff + shared_ff: behind the experts' units may lie
 // those of a shared expert that every row uses with weight 1 and a limit of its own. An expert the row does not use
 // (w = 0) gives exact zeros.
-__device__ __forceinline__ float clamped_unit(float gate, float up, float w, float limit, float alpha) {
-    const float g = fminf(__fmul_rn(w, gate), limit);
-    const float u = fminf(fmaxf(__fmul_rn(w, up), -limit), limit);
-    return __fmul_rn(g / (1.f + expf(-__fmul_rn(alpha, g))), u + 1.f);
+// With `on_output` the weight multiplies the unit's result instead, and the table has a column more for the shared expert's units.
+__device__ __forceinline__ float clamped_unit(float gate, float up, float w, float limit, float alpha, int on_output) {
+    const float wi = on_output ? 1.f : w;
+    const float g = fminf(__fmul_rn(wi, gate), limit);
+    const float u = fminf(fmaxf(__fmul_rn(wi, up), -limit), limit);
+    const float y = __fmul_rn(g / (1.f + expf(-__fmul_rn(alpha, g))), u + 1.f);
+    return on_output ? __fmul_rn(y, w) : y;
+}
+__device__ __forceinline__ float unit_weight(const float* __restrict__ weights, size_t r, int col, int routed, int experts, int ff,
+                                             int ld_w, int on_output) {
+    if (weights == nullptr) return 1.f;
+    if (col < routed) return weights[r * ld_w + col / ff];
+    return on_output && ld_w > experts ? weights[r * ld_w + experts] : 1.f;
 }
 
 template <typename T>
 __global__ void glu_clamped_kernel(const T* __restrict__ gate_up, const float* __restrict__ weights, T* __restrict__ out,
                                    int experts, int ff, float limit, int shared_ff, float shared_limit, float alpha,
-                                   size_t total) {
+                                   size_t total, int ld_w, int on_output) {
     pdl_wait();
     pdl_trigger();
     const size_t routed = (size_t)experts * ff, width = routed + shared_ff;
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
         const size_t r = i / width, col = i - r * width;
         const bool own = col < routed;
-        const float w = own && weights ? weights[r * experts + col / ff] : 1.f;
+        const float w = unit_weight(weights, r, (int)col, (int)routed, experts, ff, ld_w, on_output);
         const T* row = gate_up + r * 2 * width;
-        out[i] = from_float<T>(clamped_unit(to_float(row[col]), to_float(row[width + col]), w, own ? limit : shared_limit, alpha));
+        out[i] = from_float<T>(clamped_unit(to_float(row[col]), to_float(row[width + col]), w, own ? limit : shared_limit, alpha, on_output));
     }
 }
 
@@ -172,7 +182,7 @@ __global__ void glu_clamped_kernel(const T* __restrict__ gate_up, const float* _
 template <typename T>
 __global__ void __launch_bounds__(256)
 glu_clamped_vec_kernel(const T* __restrict__ gate_up, const float* __restrict__ weights, T* __restrict__ out, int experts, int ff,
-                       float limit, int shared_ff, float shared_limit, float alpha, int rows) {
+                       float limit, int shared_ff, float shared_limit, float alpha, int rows, int ld_w, int on_output) {
     constexpr int N = 16 / sizeof(T);
     pdl_wait();
     pdl_trigger();
@@ -184,7 +194,7 @@ glu_clamped_vec_kernel(const T* __restrict__ gate_up, const float* __restrict__ 
     for (int gi = blockIdx.x * blockDim.x + threadIdx.x; gi < groups; gi += gridDim.x * blockDim.x) {
         const int col = gi * N;
         const bool own = col < routed;
-        const float w = own && weights ? weights[(size_t)r * experts + col / ff] : 1.f;
+        const float w = unit_weight(weights, r, col, routed, experts, ff, ld_w, on_output);
         uint4 res;
         T* y = reinterpret_cast<T*>(&res);
         if (w == 0.f) {         // the row does not use this expert: its units are not read
@@ -196,7 +206,7 @@ glu_clamped_vec_kernel(const T* __restrict__ gate_up, const float* __restrict__ 
             const T* u = reinterpret_cast<const T*>(&uraw);
             const float lim = own ? limit : shared_limit;
 #pragma unroll
-            for (int k = 0; k < N; ++k) y[k] = from_float<T>(clamped_unit(to_float(g[k]), to_float(u[k]), w, lim, alpha));
+            for (int k = 0; k < N; ++k) y[k] = from_float<T>(clamped_unit(to_float(g[k]), to_float(u[k]), w, lim, alpha, on_output));
         }
         *reinterpret_cast<uint4*>(dst + col) = res;
     }
@@ -205,9 +215,11 @@ glu_clamped_vec_kernel(const T* __restrict__ gate_up, const float* __restrict__ 
 }  // namespace
 
 // gate_up [rows, 2 * (experts * ff + shared_ff)], out [rows, experts * ff + shared_ff], both contiguous and of type
-// `dtype`; weights [rows, experts] float32 or null.
+// `dtype`; weights [rows, ld_w] float32 or null (`on_output`: they multiply the units' results, a shared
+// expert's by column `experts`).
 JLLM_EXPORT int jllm_glu_clamped(const void* gate_up, const float* weights, void* out, int dtype, int rows, int experts, int ff,
-                                 float limit, int shared_ff, float shared_limit, float alpha, cudaStream_t stream) {
+                                 float limit, int shared_ff, float shared_limit, float alpha, int ld_w, int on_output,
+                                 cudaStream_t stream) {
     JLLM_REQUIRE(rows >= 0 && experts > 0 && ff > 0 && limit > 0.f && shared_ff >= 0 && (shared_ff == 0 || shared_limit > 0.f),
                  "glu_clamped: rows=%d experts=%d ff=%d limit=%g shared_ff=%d shared_limit=%g", rows, experts, ff, (double)limit,
                  shared_ff, (double)shared_limit);
@@ -218,30 +230,30 @@ JLLM_EXPORT int jllm_glu_clamped(const void* gate_up, const float* weights, void
         const dim3 grid(max(1, min(64, (width / per + 255) / 256)), rows);
         if (dtype == JLLM_F32)
             jllm_launch(glu_clamped_vec_kernel<float>, grid, dim3(256), 0, stream, LAUNCH_DEPENDENT, (const float*)gate_up, weights,
-                        (float*)out, experts, ff, limit, shared_ff, shared_limit, alpha, rows);
+                        (float*)out, experts, ff, limit, shared_ff, shared_limit, alpha, rows, ld_w, on_output);
         else
             jllm_launch(glu_clamped_vec_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, LAUNCH_DEPENDENT,
                         (const __nv_bfloat16*)gate_up, weights, (__nv_bfloat16*)out, experts, ff, limit, shared_ff, shared_limit,
-                        alpha, rows);
+                        alpha, rows, ld_w, on_output);
         return jllm_check_launch("glu_clamped");
     }
     const size_t total = (size_t)rows * width;
     const int blocks = (int)min((size_t)65535, (total + 255) / 256);
     if (dtype == JLLM_F32)
         jllm_launch(glu_clamped_kernel<float>, dim3(blocks), dim3(256), 0, stream, LAUNCH_DEPENDENT, (const float*)gate_up, weights,
-                    (float*)out, experts, ff, limit, shared_ff, shared_limit, alpha, total);
+                    (float*)out, experts, ff, limit, shared_ff, shared_limit, alpha, total, ld_w, on_output);
     else
         jllm_launch(glu_clamped_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, LAUNCH_DEPENDENT,
                     (const __nv_bfloat16*)gate_up, weights, (__nv_bfloat16*)out, experts, ff, limit, shared_ff, shared_limit, alpha,
-                    total);
+                    total, ld_w, on_output);
     return jllm_check_launch("glu_clamped");
 }
 
 // h [rows, ld] of type `dtype` (the normed rows); router [experts + identity + gates, dim] float32; correction
-// [experts + identity] or null; weights [rows, ld_out] float32: the experts' weights, then the gates, then (with identity
+// [experts + identity] or null; bias likewise; weights [rows, ld_out] float32: the experts' weights, then the gates, then (with identity
 // entries) the sum of the chosen identity entries' weights.
-JLLM_EXPORT int jllm_route_experts(const void* h, int dtype, int ld, const float* router, const void* correction,
-                                   int correction_dtype, float* weights, int rows, int dim, int real, int top, float scale,
+JLLM_EXPORT int jllm_route_experts(const void* h, int dtype, int ld, const float* router, const void* bias, int bias_dtype,
+                                   const void* correction, int correction_dtype, float* weights, int rows, int dim, int real, int top, float scale,
                                    int normalize, int identity, int gates, int softmax, int ld_out, cudaStream_t stream) {
     const int experts = real + identity + gates;
     JLLM_REQUIRE(rows >= 0 && dim > 0 && real > 0 && identity >= 0 && gates >= 0 && top >= 1 && top <= real + identity &&
@@ -249,7 +261,7 @@ JLLM_EXPORT int jllm_route_experts(const void* h, int dtype, int ld, const float
                  "route_experts: rows=%d dim=%d experts=%d identity=%d gates=%d top=%d ld_out=%d", rows, dim, real, identity, gates,
                  top, ld_out);
     if (rows == 0) return JLLM_OK;
-    const VecRef c{correction, correction_dtype};
+    const VecRef c{correction, correction_dtype}, lb{bias, bias_dtype};
     const int padded = (experts + 1) / 2 * 2;       // the row's copy behind the two score arrays starts on 16 bytes
     const size_t smem = (2 * (size_t)padded + ((dim + 3) & ~3) + ld_out) * sizeof(float);
     JLLM_REQUIRE(smem <= 200 * 1024, "route_experts: dim=%d and experts=%d need %zu bytes of shared memory", dim, experts, smem);
@@ -260,10 +272,10 @@ JLLM_EXPORT int jllm_route_experts(const void* h, int dtype, int ld, const float
     }
     if (dtype == JLLM_F32)
         jllm_launch(route_experts_kernel<float>, dim3(rows), dim3(256), smem, stream, LAUNCH_DEPENDENT, (const float*)h, ld,
-                    router, c, (int)(correction != nullptr), weights, dim, real, top, scale, normalize, identity, gates, softmax, ld_out);
+                    router, lb, (int)(bias != nullptr), c, (int)(correction != nullptr), weights, dim, real, top, scale, normalize, identity, gates, softmax, ld_out);
     else
         jllm_launch(route_experts_kernel<__nv_bfloat16>, dim3(rows), dim3(256), smem, stream, LAUNCH_DEPENDENT,
-                    (const __nv_bfloat16*)h, ld, router, c, (int)(correction != nullptr), weights, dim, real, top, scale,
+                    (const __nv_bfloat16*)h, ld, router, lb, (int)(bias != nullptr), c, (int)(correction != nullptr), weights, dim, real, top, scale,
                     normalize, identity, gates, softmax, ld_out);
     return jllm_check_launch("route_experts");
 }

@@ -13,7 +13,8 @@ constexpr int BULK_WARP_BYTES = 32 * 32 * 4;                // ... and for `bulk
 template <typename Tout>
 struct TileEpilogue {
     Tout* out;
-    int ldo, M, N, accumulate, has_bias, swiglu;
+    int ldo, M, N, accumulate, has_bias;
+    GluArgs swiglu;
     VecRef bias;
     // not null: a float32 output written (or added into) by tiled bulk copies of 32 x 32 blocks from shared memory,
     // which the copy engine clips to [M, N]; the residual add is then done where the data lies (in L2), the SM neither
@@ -111,11 +112,19 @@ struct TileEpilogue {
             Tout* dst = out + (size_t)row * ldo + (n_base >> 1);
             // (the tensor-core path may use the fast exponential: its result is rounded to bfloat16 anyway)
             float hv[16];
+            const int unit0 = n_base >> 1;
+            const bool weighted = swiglu.weights != nullptr, eights = swiglu.in_eights();
+            float wt[2] = {1.f, 1.f};
+            if (weighted && eights) {
+                wt[0] = swiglu.weight(row, unit0);
+                wt[1] = swiglu.weight(row, unit0 + 8);
+            }
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
                 const int cg = (j >> 3) * 16 + (j & 7);
                 const float gt = __uint_as_float(v[cg]), up = __uint_as_float(v[cg + 8]);
-                hv[j] = glu_unit<true>(gt, up, swiglu);
+                hv[j] = glu_unit<true>(gt, up, swiglu.word_of(unit0 + j));
+                if (weighted) hv[j] = __fmul_rn(hv[j], eights ? wt[j >> 3] : swiglu.weight(row, unit0 + j));
             }
             if (sizeof(Tout) == 2 && n_base + 32 <= N && ((((uintptr_t)dst) & 15u) == 0)) {
                 uint32_t p[8];

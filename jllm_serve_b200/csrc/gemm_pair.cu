@@ -90,7 +90,7 @@ template <typename Tout>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(THREADS, 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                  const __grid_constant__ CUtensorMap map_out, int bulk_out, VecRef bias,
-                 int has_bias, Tout* __restrict__ out, int ldo, int accumulate, int M, int N, int K, int swiglu,
+                 int has_bias, Tout* __restrict__ out, int ldo, int accumulate, int M, int N, int K, GluArgs swiglu,
                  int stream, float* __restrict__ partials, int* __restrict__ counters, int* __restrict__ error_word) {
     extern __shared__ uint8_t smem_raw[];
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;   // swizzled tiles want 1024-byte alignment
@@ -473,8 +473,9 @@ JLLM_EXPORT int jllm_gemm_pair_fits(const void* a, int lda, const void* w_packed
 // w: ops.pack_weight of the [N, K] weight (k_blocks_packed = ceil(K / 64) its k blocks).
 JLLM_EXPORT int jllm_gemm_pair(const void* a, int lda, const void* w, int k_blocks_packed, const void* bias, int bias_dtype,
                                void* out, int out_dtype, int ldo, int accumulate, int M, int N, int K, int max_pairs,
-                               int swiglu, float* workspace, long long workspace_floats, int stream_mode,
+                               int swiglu_word, const void* glu_more, float* workspace, long long workspace_floats, int stream_mode,
                                cudaStream_t stream) {
+    const GluArgs swiglu = glu_args(swiglu_word, glu_more);
     JLLM_REQUIRE(jllm_gemm_pair_fits(a, lda, w, M, N, K),
                  "gemm_pair: needs K %% 8 == 0 and 16-byte aligned rows (M=%d N=%d K=%d lda=%d)", M, N, K, lda);
     JLLM_REQUIRE(k_blocks_packed == (K + BK - 1) / BK, "gemm_pair: the packed weight has %d k blocks, K=%d needs %d",

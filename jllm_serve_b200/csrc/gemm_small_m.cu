@@ -49,7 +49,7 @@ template <int NT, int RT, int UNROLL, typename Tout>
 __global__ void __launch_bounds__(WARPS * 32, 2)
 gemm_small_m_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfloat16* __restrict__ w, int k_blocks,
                     VecRef bias, int has_bias, Tout* __restrict__ out, int ldo, int accumulate, int M, int N, int K,
-                    int swiglu) {
+                    GluArgs swiglu) {
     extern __shared__ float red[];  // [WARPS][RT * 16][NT * 8]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
@@ -168,7 +168,7 @@ gemm_small_m_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfl
             float u = 0.f;
 #pragma unroll
             for (int wi = 0; wi < WARPS; ++wi) u += red[(size_t)wi * ROWS * TOK + e + 8];
-            out[(size_t)tok * ldo + (n >> 4) * 8 + (row & 7)] = from_float<Tout>(glu_unit<false>(v, u, swiglu));
+            out[(size_t)tok * ldo + (n >> 4) * 8 + (row & 7)] = from_float<Tout>(swiglu.apply<false>(v, u, tok, (n >> 4) * 8 + (row & 7)));
             continue;
         }
         if (has_bias) v += bias[n];
@@ -181,7 +181,7 @@ gemm_small_m_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfl
 
 template <int NT, int RT, int UNROLL>
 int launch(const void* a, int lda, const void* w, int k_blocks, VecRef bias, int has_bias, void* out, int out_dtype, int ldo,
-           int accumulate, int M, int N, int K, int swiglu, cudaStream_t stream) {
+           int accumulate, int M, int N, int K, GluArgs swiglu, cudaStream_t stream) {
     const int grid = (N + 16 * RT - 1) / (16 * RT);
     const size_t smem = (size_t)WARPS * RT * 16 * NT * 8 * sizeof(float);
     if (out_dtype == JLLM_F32) {
@@ -209,7 +209,8 @@ JLLM_EXPORT int jllm_gemm_small_m_fits(const void* a, int lda, const void* w_pac
 // w_packed: ops.pack_weight of the [N, K] weight, k_blocks = ceil(K / 64) its k blocks.
 JLLM_EXPORT int jllm_gemm_small_m(const void* a, int lda, const void* w, int k_blocks, const void* bias, int bias_dtype,
                                   void* out, int out_dtype, int ldo, int accumulate, int M, int N, int K,
-                                  int swiglu, cudaStream_t stream) {
+                                  int swiglu_word, const void* glu_more, cudaStream_t stream) {
+    const GluArgs swiglu = glu_args(swiglu_word, glu_more);
     JLLM_REQUIRE(jllm_gemm_small_m_fits(a, lda, w, M, N, K),
                  "gemm_small_m: needs 1 <= M <= 64, K %% 8 == 0 and 16-byte aligned rows (M=%d N=%d K=%d lda=%d)",
                  M, N, K, lda);

@@ -44,7 +44,7 @@ __device__ __forceinline__ void tmem_ld_32x32b_x16(uint32_t taddr, uint32_t (&r)
 template <typename Tout>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_stream_kernel(const __grid_constant__ CUtensorMap map_a, const __nv_bfloat16* __restrict__ w_packed, VecRef bias,
-                   int has_bias, Tout* __restrict__ out, int ldo, int accumulate, int M, int N, int k_blocks, int swiglu,
+                   int has_bias, Tout* __restrict__ out, int ldo, int accumulate, int M, int N, int k_blocks, GluArgs swiglu,
                    int ntok, int stages, uint32_t tmem_cols, float* __restrict__ partials,
                    int* __restrict__ counters, int* __restrict__ error_word) {
     extern __shared__ uint8_t smem_raw[];
@@ -185,7 +185,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_a, const __nv_bfloat1
                         const float other = __shfl_xor_sync(0xffffffffu, v[j], 8);
                         if ((lane & 8) == 0 && n + 8 < N && m0 + j < M) {
                             const float gt = v[j];
-                            out[(size_t)(m0 + j) * ldo + unit] = from_float<Tout>(glu_unit<true>(gt, other, swiglu));
+                            out[(size_t)(m0 + j) * ldo + unit] = from_float<Tout>(swiglu.apply<true>(gt, other, m0 + j, unit));
                         }
                     }
                 } else if (n < N) {
@@ -325,8 +325,9 @@ JLLM_EXPORT long long jllm_gemm_stream_workspace_floats() { return 2LL * MAX_TIL
 // (counters, then parked parts), at least jllm_gemm_stream_workspace_floats().
 JLLM_EXPORT int jllm_gemm_stream(const void* a, int lda, const void* w_packed, int k_blocks, const void* bias,
                                  int bias_dtype, void* out, int out_dtype, int ldo, int accumulate, int M, int N, int K,
-                                 int swiglu, float* workspace, long long workspace_floats, int max_blocks,
+                                 int swiglu_word, const void* glu_more, float* workspace, long long workspace_floats, int max_blocks,
                                  cudaStream_t stream) {
+    const GluArgs swiglu = glu_args(swiglu_word, glu_more);
     JLLM_REQUIRE(M >= 1 && M <= MAX_TOKENS && N >= 1 && K >= 8 && K % 8 == 0 && lda % 8 == 0 && ((uintptr_t)a % 16) == 0 &&
                      ((uintptr_t)w_packed % 16) == 0,
                  "gemm_stream: needs 1 <= rows <= %d, K %% 8 == 0 and 16-byte aligned rows and weights "

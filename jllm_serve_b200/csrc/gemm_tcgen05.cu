@@ -52,7 +52,7 @@ template <typename Tout, int BN>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_out, int bulk_out,
                     const __nv_bfloat16* __restrict__ w_packed, VecRef bias,
-                    int has_bias, Tout* __restrict__ out, int ldo, int accumulate, int M, int N, int K, int swiglu,
+                    int has_bias, Tout* __restrict__ out, int ldo, int accumulate, int M, int N, int K, GluArgs swiglu,
                     int stream, float* __restrict__ partials, int* __restrict__ counters, int* __restrict__ error_word,
                     int starve) {
     // `starve` (a test of the bounded waits, never set otherwise): the first stage's barrier expects 16 bytes more than
@@ -372,8 +372,9 @@ JLLM_EXPORT void jllm_gemm_plain_stores(int on) { g_plain_stores = on; }
 // w: ops.pack_weight of the [N, K] weight (k_blocks_packed = ceil(K / 64) its k blocks).
 JLLM_EXPORT int jllm_gemm_tcgen05(const void* a, int lda, const void* w, int k_blocks_packed, const void* bias, int bias_dtype,
                                   void* out, int out_dtype, int ldo, int accumulate, int M, int N, int K, int max_blocks,
-                                  int swiglu, float* workspace, long long workspace_floats, int stream_mode,
+                                  int swiglu_word, const void* glu_more, float* workspace, long long workspace_floats, int stream_mode,
                                   int tile_width, cudaStream_t stream) {
+    const GluArgs swiglu = glu_args(swiglu_word, glu_more);
     JLLM_REQUIRE(jllm_gemm_tcgen05_fits(a, lda, w, M, N, K),
                  "gemm_tcgen05: needs K %% 8 == 0 and 16-byte aligned rows (M=%d N=%d K=%d lda=%d)", M, N, K, lda);
     JLLM_REQUIRE(k_blocks_packed == (K + BK - 1) / BK, "gemm_tcgen05: the packed weight has %d k blocks, K=%d needs %d",

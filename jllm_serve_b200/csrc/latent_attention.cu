@@ -14,7 +14,7 @@
 //                       latent-space query (where `gemm_heads` put it), so that one dot product with a cached row gives
 //                       both terms of the score
 //   gemm_heads          out[r, h, :] = f(r, h) * W[h] a[r, h, :] for every head h at once (W [heads, N, K]); f = alpha, or
-//                       alpha * sigmoid(gate[r, h]) (the mixer's output gate). float32: on the CUDA cores with one
+//                       alpha * sigmoid(gate[r, h]) (the mixer's output gate; one per head, or one per value of a head). float32: on the CUDA cores with one
 //                       accumulator per element in ascending k. bfloat16: 64 x 64 tiles per (head, block) on the tensor
 //                       cores (mma.sync m16n8k16, float32 accumulation), operands staged in shared memory 32 k at a
 //                       time. Either way a row's result depends on that row alone, not on the batch.
@@ -25,7 +25,7 @@ namespace {
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_norm_store_kernel(const T* __restrict__ src, int ld, VecRef gain, const int* __restrict__ slots, T* __restrict__ cache,
-                         int rank, float eps, long long cache_rows) {
+                         int rank, int width, float eps, long long cache_rows) {
     __shared__ float scratch[33];
     pdl_wait();
     pdl_trigger();
@@ -40,9 +40,10 @@ latent_norm_store_kernel(const T* __restrict__ src, int ld, VecRef gain, const i
     const float inv = 1.f / sqrtf(ss / (float)rank + eps);
     const int slot = slots[r];
     if (!jllm_in_bounds(slot, cache_rows, BOUNDS_SLOT)) return;
-    T* dst = cache + (size_t)slot * rank;
+    T* dst = cache + (size_t)slot * width;
     for (int i = threadIdx.x; i < rank; i += blockDim.x)
         dst[i] = from_float<T>(__fmul_rn(__fmul_rn(to_float(row[i]), inv), gain[i]));
+    for (int i = rank + threadIdx.x; i < width; i += blockDim.x) dst[i] = from_float<T>(0.f);
 }
 
 // Turns neighbouring pairs: (u, v) -> (u cos - v sin, v cos + u sin), the angle of pair i from the position's table row.
@@ -159,7 +160,7 @@ constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;
 template <typename T>
 __global__ void __launch_bounds__(256)
 gemm_heads_kernel(const T* __restrict__ a, int lda, const T* __restrict__ w, T* __restrict__ out, int ldo,
-                  const T* __restrict__ gate, int ld_gate, float alpha, int M, int N, int K, int a_head, int o_head, HeadRope rp) {
+                  const T* __restrict__ gate, int ld_gate, int gate_full, float alpha, int M, int N, int K, int a_head, int o_head, HeadRope rp) {
     __shared__ float as[BK][BM + 4];
     __shared__ float ws[BK][BN + 4];
     pdl_wait();
@@ -203,14 +204,18 @@ gemm_heads_kernel(const T* __restrict__ a, int lda, const T* __restrict__ w, T* 
         const int m = m0 + ty * TM + i;
         if (m >= M) continue;
         float f = alpha;
-        if (gate != nullptr) {
+        if (gate != nullptr && !gate_full) {
             const float gv = to_float(gate[(size_t)m * ld_gate + h]);
             f = __fmul_rn(alpha, 1.f / (1.f + expf(-gv)));
         }
 #pragma unroll
         for (int j = 0; j < TN; ++j) {
             const int n = n0 + tx * TN + j;
-            if (n < N) out[(size_t)m * ldo + (size_t)h * o_head + n] = from_float<T>(__fmul_rn(acc[i][j], f));
+            if (n < N) {
+                float fn = f;
+                if (gate_full) fn = __fmul_rn(f, 1.f / (1.f + expf(-to_float(gate[(size_t)m * ld_gate + (size_t)h * N + n]))));
+                out[(size_t)m * ldo + (size_t)h * o_head + n] = from_float<T>(__fmul_rn(acc[i][j], fn));
+            }
         }
     }
 }
@@ -231,7 +236,7 @@ template <bool VEC>
 __global__ void __launch_bounds__(128)
 gemm_heads_mma_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfloat16* __restrict__ w,
                       __nv_bfloat16* __restrict__ out, int ldo, const __nv_bfloat16* __restrict__ gate, int ld_gate,
-                      float alpha, int M, int N, int K, int a_head, int o_head, HeadRope rp) {
+                      int gate_full, float alpha, int M, int N, int K, int a_head, int o_head, HeadRope rp) {
     __shared__ __align__(16) __nv_bfloat16 as[64][HPAD];
     __shared__ __align__(16) __nv_bfloat16 ws[64][HPAD];
     pdl_wait();
@@ -289,7 +294,7 @@ gemm_heads_mma_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_b
         const int m = m0 + warp * 16 + g + 8 * half;
         if (m >= M) continue;
         float f = alpha;
-        if (gate != nullptr) {
+        if (gate != nullptr && !gate_full) {
             const float gv = to_float(gate[(size_t)m * ld_gate + h]);
             f = __fmul_rn(alpha, 1.f / (1.f + expf(-gv)));
         }
@@ -297,8 +302,14 @@ gemm_heads_mma_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_b
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
             const int n = n0 + 8 * j + 2 * t;
-            if (n < N) dst[n] = __float2bfloat16_rn(__fmul_rn(acc[j][2 * half], f));
-            if (n + 1 < N) dst[n + 1] = __float2bfloat16_rn(__fmul_rn(acc[j][2 * half + 1], f));
+            float f0 = f, f1 = f;
+            if (gate_full) {
+                const __nv_bfloat16* gm = gate + (size_t)m * ld_gate + (size_t)h * N + n;
+                if (n < N) f0 = __fmul_rn(f, 1.f / (1.f + expf(-__bfloat162float(gm[0]))));
+                if (n + 1 < N) f1 = __fmul_rn(f, 1.f / (1.f + expf(-__bfloat162float(gm[1]))));
+            }
+            if (n < N) dst[n] = __float2bfloat16_rn(__fmul_rn(acc[j][2 * half], f0));
+            if (n + 1 < N) dst[n + 1] = __float2bfloat16_rn(__fmul_rn(acc[j][2 * half + 1], f1));
         }
     }
 }
@@ -307,27 +318,28 @@ gemm_heads_mma_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_b
 
 JLLM_BOUNDS_READER(latent_attention)
 
-// src [rows, ld] (the down-projected rows), cache [cache_rows, rank] (a page pool seen as rows: slot = page * page_size
+// src [rows, ld] (the down-projected rows), cache [cache_rows, width] (zeros behind the rank values; a page pool seen as rows: slot = page * page_size
 // + offset), both of type `dtype`.
 JLLM_EXPORT int jllm_latent_norm_store(const void* src, int dtype, int ld, const void* gain, int gain_dtype,
-                                       const int* slots, void* cache, long long cache_rows, int rows, int rank, float eps,
+                                       const int* slots, void* cache, long long cache_rows, int rows, int rank, int width, float eps,
                                        cudaStream_t stream) {
-    JLLM_REQUIRE(rows >= 0 && rank > 0 && ld >= rank, "latent_norm_store: rows=%d rank=%d ld=%d", rows, rank, ld);
+    JLLM_REQUIRE(rows >= 0 && rank > 0 && ld >= rank && width >= rank, "latent_norm_store: rows=%d rank=%d ld=%d", rows, rank, ld);
     if (rows == 0) return JLLM_OK;
     const VecRef g{gain, gain_dtype};
     if (dtype == JLLM_F32)
         jllm_launch(latent_norm_store_kernel<float>, dim3(rows), dim3(128), 0, stream, LAUNCH_DEPENDENT, (const float*)src,
-                    ld, g, slots, (float*)cache, rank, eps, cache_rows);
+                    ld, g, slots, (float*)cache, rank, width, eps, cache_rows);
     else
         jllm_launch(latent_norm_store_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, stream, LAUNCH_DEPENDENT,
-                    (const __nv_bfloat16*)src, ld, g, slots, (__nv_bfloat16*)cache, rank, eps, cache_rows);
+                    (const __nv_bfloat16*)src, ld, g, slots, (__nv_bfloat16*)cache, rank, width, eps, cache_rows);
     return jllm_check_launch("latent_norm_store");
 }
 
 // a [M, lda] with head h's K values at column h * a_head (0: h * K); w [heads, N, K]; out [M, ldo] with head h's N values at
-// h * o_head (0: h * N); gate (or null) [M, ld_gate] with head h's gate at column h.
+// h * o_head (0: h * N); gate (or null) [M, ld_gate] with head h's gate at column h, or (`gate_full`) the gate of its n-th value at
+// column h * N + n.
 JLLM_EXPORT int jllm_gemm_heads(const void* a, int dtype, int lda, const void* w, void* out, int ldo, const void* gate,
-                                int ld_gate, float alpha, int M, int heads, int N, int K, int a_head, int o_head, int rope_dim,
+                                int ld_gate, int gate_full, float alpha, int M, int heads, int N, int K, int a_head, int o_head, int rope_dim,
                                 const float* cos_t, const float* sin_t, int rotary_dim, const int* positions,
                                 cudaStream_t stream) {
     JLLM_REQUIRE(M >= 0 && heads > 0 && N > 0 && K > 0, "gemm_heads: M=%d heads=%d N=%d K=%d", M, heads, N, K);
@@ -345,16 +357,16 @@ JLLM_EXPORT int jllm_gemm_heads(const void* a, int dtype, int lda, const void* w
     static_assert(BM == 64 && BN == 64, "both kernels take 64 x 64 tiles");
     if (dtype == JLLM_F32) {
         jllm_launch(gemm_heads_kernel<float>, grid, dim3(256), 0, stream, LAUNCH_DEPENDENT, (const float*)a, lda,
-                    (const float*)w, (float*)out, ldo, (const float*)gate, ld_gate, alpha, M, N, K, a_head, o_head, rp);
+                    (const float*)w, (float*)out, ldo, (const float*)gate, ld_gate, gate != nullptr && gate_full, alpha, M, N, K, a_head, o_head, rp);
         return jllm_check_launch("gemm_heads");
     }
     const bool vec = K % 8 == 0 && lda % 8 == 0 && a_head % 8 == 0 && ((uintptr_t)a % 16) == 0 && ((uintptr_t)w % 16) == 0;
     if (vec)
         jllm_launch(gemm_heads_mma_kernel<true>, grid, dim3(128), 0, stream, LAUNCH_DEPENDENT, (const __nv_bfloat16*)a, lda,
-                    (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, (const __nv_bfloat16*)gate, ld_gate, alpha, M, N, K, a_head, o_head, rp);
+                    (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, (const __nv_bfloat16*)gate, ld_gate, gate != nullptr && gate_full, alpha, M, N, K, a_head, o_head, rp);
     else
         jllm_launch(gemm_heads_mma_kernel<false>, grid, dim3(128), 0, stream, LAUNCH_DEPENDENT, (const __nv_bfloat16*)a, lda,
-                    (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, (const __nv_bfloat16*)gate, ld_gate, alpha, M, N, K, a_head, o_head, rp);
+                    (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, (const __nv_bfloat16*)gate, ld_gate, gate != nullptr && gate_full, alpha, M, N, K, a_head, o_head, rp);
     return jllm_check_launch("gemm_heads");
 }
 

@@ -134,24 +134,24 @@ class _Signatures:
     jllm_swiglu = [P, P, I, I, I, I, P]
     jllm_qk_norm_rope_store = [P, I, P, P, I, I, F, P, P, I, P, P, P, P, I, I, I, I, I, I, I, P]
     jllm_gemm_plain = [P, I, I, P, I, P, I, P, I, I, I, I, I, I, P]
-    jllm_gemm_small_m = [P, I, P, I, P, I, P, I, I, I, I, I, I, I, P]
-    jllm_gemm_tcgen05 = [P, I, P, I, P, I, P, I, I, I, I, I, I, I, I, P, ctypes.c_longlong, I, I, P]
-    jllm_gemm_pair = [P, I, P, I, P, I, P, I, I, I, I, I, I, I, I, P, ctypes.c_longlong, I, P]
+    jllm_gemm_small_m = [P, I, P, I, P, I, P, I, I, I, I, I, I, I, P, P]
+    jllm_gemm_tcgen05 = [P, I, P, I, P, I, P, I, I, I, I, I, I, I, I, P, P, ctypes.c_longlong, I, I, P]
+    jllm_gemm_pair = [P, I, P, I, P, I, P, I, I, I, I, I, I, I, I, P, P, ctypes.c_longlong, I, P]
     jllm_gemm_pair_resident = []
     jllm_gemm_plain_stores = [I]
-    jllm_gemm_stream = [P, I, P, I, P, I, P, I, I, I, I, I, I, I, P, ctypes.c_longlong, I, P]
+    jllm_gemm_stream = [P, I, P, I, P, I, P, I, I, I, I, I, I, I, P, P, ctypes.c_longlong, I, P]
     jllm_gemm_tcgen05_error = []
     jllm_gemm_tcgen05_starve_next = []
-    jllm_attention_plain = [P, I, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P, I, P]
+    jllm_attention_plain = [P, I, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P, I, F, P]
     jllm_attention_decode = [P, I, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, I, P, P]
-    jllm_attention_decode_flat = [P, I, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, I, P, P]
-    jllm_attention_decode_extras = [P, I, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, I, P, I, P, I, P]
-    jllm_attention_prefill_extras = [P, I, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, I, P]
-    jllm_attention_prefill_tc_extras = [P, I, P, P, ctypes.c_longlong, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, I, P]
+    jllm_attention_decode_flat = [P, I, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, I, P, F, P]
+    jllm_attention_decode_extras = [P, I, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, I, P, I, P, I, F, P]
+    jllm_attention_prefill_extras = [P, I, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, I, F, P]
+    jllm_attention_prefill_tc_extras = [P, I, P, P, ctypes.c_longlong, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, I, F, P]
     jllm_attention_prefill = [P, I, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, P]
     jllm_attention_prefill_tc = [P, I, P, P, ctypes.c_longlong, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, P]
     jllm_attention_prefill_tc_error = []
-    jllm_attention_prefill_pair = [P, I, P, P, ctypes.c_longlong, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, P]
+    jllm_attention_prefill_pair = [P, I, P, P, ctypes.c_longlong, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P]
     jllm_attention_decode_separate_combine = [I]
     jllm_attention_decode_fresh = [P, I, P, P, I, I, F, P, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P]
     jllm_argmax = [P, I, I, I, P, P]
@@ -167,19 +167,21 @@ class _Signatures:
     jllm_head_gate = [P, I, I, P, I, I, I, I, P]
     jllm_norm_sum = [P, P, P, P, P, I, I, I, F, F, I, P]
     jllm_norm_chain = [P, P, P, P, P, F, P, P, P, I, I, I, I, F, P]
-    jllm_latent_norm_store = [P, I, I, P, I, P, P, ctypes.c_longlong, I, I, F, P]
-    jllm_gemm_heads = [P, I, I, P, P, I, P, I, F, I, I, I, I, I, I, I, P, P, I, P, P]
+    jllm_latent_norm_store = [P, I, I, P, I, P, P, ctypes.c_longlong, I, I, I, F, P]
+    jllm_gemm_heads = [P, I, I, P, P, I, P, I, I, F, I, I, I, I, I, I, I, P, P, I, P, P]
     jllm_latent_prepare = [P, I, I, I, P, P, I, I, I, P, I, P, P, I, P, P, P, I, ctypes.c_longlong, I, F, I, P]
     jllm_rope_heads = [P, I, I, I, I, P, I, I, I, I, I, I, P, P, I, P, P]
-    jllm_glu_clamped = [P, P, P, I, I, I, I, F, I, F, F, P]
+    jllm_glu_clamped = [P, P, P, I, I, I, I, F, I, F, F, I, I, P]
     jllm_bounds_error_residual_paths = [P]
     jllm_layernorm = [P, P, I, P, I, P, I, I, F, I, F, P]
     jllm_norm_add = [P, P, P, I, P, I, I, I, F, I, P]
     jllm_token_shift = [P, P, I, P, I, P, P, P, P, P, I, I, I, I, I, P]
     jllm_depth_mix = [P, ctypes.c_longlong, P, I, I, P, ctypes.c_longlong, P]
     jllm_scale_values = [P, F, ctypes.c_longlong, P]
+    jllm_softcap_values = [P, F, ctypes.c_longlong, P]
+    jllm_stream_mix = [P, I, P, P, P, P, P, I, P, I, P, I, I, F, I, P]
     jllm_norm_add_mix = [P, P, P, I, I, I, F, I, P, ctypes.c_longlong, P, I, I, P, P, I, P, I, P, P, P, I, P]
-    jllm_route_experts = [P, I, I, P, P, I, P, I, I, I, I, F, I, I, I, I, I, P]
+    jllm_route_experts = [P, I, I, P, P, I, P, I, P, I, I, I, I, F, I, I, I, I, I, P]
     jllm_scale_expert_hidden = [P, I, P, I, I, I, I, I, P]
     jllm_bounds_error_gated_recurrence = [P]
     jllm_ssm_gates = [P, I, P, P, I, P, P, I, I, P]
@@ -194,7 +196,7 @@ class _Signatures:
     jllm_add_rows_scaled = [P, P, I, I, P, I, I, I, P]
     jllm_norm_conv = [P, P, I, P, I, P, I, P, P, P, P, P, I, I, I, I, I, F, I, P]
     jllm_bounds_error_attention_maps = [P]
-    jllm_map_prepare = [P, I, I, I, I, P, P, F, P, P, I, I, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, P]
+    jllm_map_prepare = [P, I, I, I, I, P, P, F, P, P, I, I, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, F, P]
     jllm_map_difference = [P, I, I, I, F, F, F, P, I, I, I, I, P]
     jllm_bounds_error_delta_recurrence = [P]
     jllm_delta_tanh = [P, I, P, I, I, I, P]
@@ -311,16 +313,17 @@ def gated_head_norm(o, gate, gain, eps, scale, out, heads, value_dim, gate_kind:
 
 
 def latent_norm_store(src, gain, eps, slots, cache) -> None:
-    """cache row slots[r] = rmsnorm(src[r]) * gain; src a view [rows, rank]; cache [pages, 1, page_size, rank]."""
+    """cache row slots[r] = [rmsnorm(src[r]) * gain, zeros]; src a view [rows, rank]; cache [pages, 1, page_size, rank or more]."""
     assert src.dtype == cache.dtype and src.stride(1) == 1 and cache.is_contiguous() and slots.dtype == torch.int32
-    rank = src.shape[1]
+    rank, width = src.shape[1], cache.shape[-1]
     _call("jllm_latent_norm_store", src.data_ptr(), _DT[src.dtype], src.stride(0), gain.data_ptr(), _DT[gain.dtype],
-          slots.data_ptr(), cache.data_ptr(), cache.numel() // rank, src.shape[0], rank, float(eps), _stream())
+          slots.data_ptr(), cache.data_ptr(), cache.numel() // width, src.shape[0], rank, width, float(eps), _stream())
 
 
 def gemm_heads(a, w, out, gate=None, alpha: float = 1.0, a_head: int = 0, out_head: int = 0, rope=None) -> None:
     """out[r, h, :] = f * w[h] @ a[r, h, :] for all heads at once; a [rows, heads x K] (any row stride), w [heads, N, K]
-    contiguous, out [rows, heads x N]; f = alpha, or alpha * sigmoid(gate[r, h]) with gate a view [rows, heads]. `a_head` /
+    contiguous, out [rows, heads x N]; f = alpha, or alpha * sigmoid(gate[r, h]) with gate a view [rows, heads], or per value
+    alpha * sigmoid(gate[r, h * N + n]) with gate a view [rows, heads x N]. `a_head` /
     `out_head`: the distance between the heads of a row where it is more than K / N (a head's values are then the first K of
     every a_head values of a, and go to the first N of every out_head values of out). `rope` = (rope_dim, cos, sin, rotary_dim,
     positions): the rope_dim values behind a head's K inputs go behind its N outputs, their first rotary_dim values turned in
@@ -329,9 +332,10 @@ def gemm_heads(a, w, out, gate=None, alpha: float = 1.0, a_head: int = 0, out_he
     rope_dim, cos, sin, rotary_dim, positions = rope if rope is not None else (0, None, None, 0, None)
     assert a.dtype == w.dtype == out.dtype and w.is_contiguous() and a.stride(1) == 1 and out.stride(1) == 1
     assert a.shape[1] >= (heads - 1) * (a_head or K) + K and out.shape[1] >= (heads - 1) * (out_head or N) + N
-    assert gate is None or gate.dtype == a.dtype
+    assert gate is None or (gate.dtype == a.dtype and gate.stride(1) == 1 and gate.shape[1] in (heads, heads * N))
+    full = gate is not None and gate.shape[1] == heads * N and N > 1
     _call("jllm_gemm_heads", a.data_ptr(), _DT[a.dtype], a.stride(0), w.data_ptr(), out.data_ptr(), out.stride(0),
-          _p(gate), gate.stride(0) if gate is not None else 0, float(alpha), a.shape[0], heads, N, K, int(a_head),
+          _p(gate), gate.stride(0) if gate is not None else 0, int(full), float(alpha), a.shape[0], heads, N, K, int(a_head),
           int(out_head), int(rope_dim), _p(cos), _p(sin), int(rotary_dim), _p(positions), _stream())
 
 
@@ -366,16 +370,19 @@ SWISH_ALPHA = 1.702      # the logistic's slope in the clamped gated unit
 
 
 def glu_clamped(gate_up, weights, out, experts, ff, limit, shared_ff: int = 0, shared_limit: float = 0.0,
-                alpha: float = SWISH_ALPHA) -> None:
+                alpha: float = SWISH_ALPHA, on_output: bool = False) -> None:
     """out[r, e * ff + j] = g sigmoid(alpha g) (u + 1), g = min(w gate, limit), u = clamp(w up, -limit, limit), w =
     weights[r, e] (1 without weights); gate_up [rows, 2 x width]: all gate values, then all up values; width = experts x ff +
-    shared_ff, the last shared_ff units being a shared expert's, which every row uses with weight 1 and `shared_limit`."""
+    shared_ff, the last shared_ff units being a shared expert's, which every row uses with weight 1 and `shared_limit`.
+    `on_output`: the weights multiply the units' results and not their inputs, a shared expert's by weights[r, experts]."""
     width = experts * ff + shared_ff
     assert gate_up.dtype == out.dtype and gate_up.is_contiguous() and out.is_contiguous()
     assert gate_up.shape[1] == 2 * width and out.shape[1] == width
-    assert weights is None or (weights.dtype == torch.float32 and weights.is_contiguous() and weights.shape[1] == experts)
+    assert weights is None or (weights.dtype == torch.float32 and weights.is_contiguous()
+                                and (weights.shape[1] == experts or (on_output and weights.shape[1] > experts)))
     _call("jllm_glu_clamped", gate_up.data_ptr(), _p(weights), out.data_ptr(), _DT[out.dtype], out.shape[0], int(experts),
-          int(ff), float(limit), int(shared_ff), float(shared_limit), float(alpha), _stream())
+          int(ff), float(limit), int(shared_ff), float(shared_limit), float(alpha), weights.shape[1] if weights is not None else 0,
+          int(bool(on_output)), _stream())
 
 
 def layernorm(x, gain, eps, out, row_index=None, rows=None, center: bool = True, out_scale: float = 1.0) -> None:
@@ -459,10 +466,36 @@ def scale_values(x, s: float) -> None:
     _call("jllm_scale_values", x.data_ptr(), float(s), x.numel(), _stream())
 
 
+def softcap_values(x, cap: float) -> None:
+    """x = cap * tanh(x / cap), float32 and contiguous."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and cap > 0
+    _call("jllm_softcap_values", x.data_ptr(), float(cap), x.numel(), _stream())
+
+
+def stream_mix(streams, start=None, result=None, mix=None, read=None, gain=None, eps: float = 0.0, out=None, row_index=None,
+               rows: int | None = None, write: bool = True) -> None:
+    """A residual of several streams ([rows, S, dim] float32) between a part and the next, in one launch. `start` [rows, dim]: the
+    streams begin as copies of it. `result` [rows, dim] with `mix` (S x S values [from, to], then S): X_t = sum_s mix[s, t] X_s +
+    mix[S * S + t] result. `read` (S values): out[r] = rmsnorm(sum_s read[s] X_s) * gain in out's type; with `row_index` for the rows
+    it names only (`write` must be off). `write`: the streams are stored."""
+    n, S, dim = streams.shape
+    assert streams.dtype == torch.float32 and streams.is_contiguous()
+    assert all(t is None or (t.dtype == torch.float32 and t.is_contiguous()) for t in (start, result, mix, read))
+    assert start is None or start.shape == (n, dim)
+    assert result is None or (result.shape == (n, dim) and mix.numel() == S * S + S)
+    assert read is None or (read.numel() == S and out.is_contiguous() and out.shape[1] == dim and gain.is_contiguous())
+    count = n if row_index is None else (row_index.numel() if rows is None else rows)
+    assert out is None or out.shape[0] >= count
+    _call("jllm_stream_mix", streams.data_ptr(), S, _p(start), _p(result), _p(mix), _p(read), _p(gain),
+          _DT[gain.dtype] if gain is not None else F32, _p(out), _DT[out.dtype] if out is not None else F32, _p(row_index), count, dim,
+          float(eps), int(bool(write)), _stream())
+
+
 def route_experts(h, router, correction, top, scale, normalize, weights, identity: int = 0, gates: int = 0,
-                  softmax: bool = False) -> None:
+                  softmax: bool = False, bias=None) -> None:
     """weights[r, e] = the weight of expert e for row r (0 where it is not among the row's `top`): scores sigmoid(router
-    h) in float32 (or, with `softmax`, the softmax of router h over all entries), choice by score + correction, chosen
+    h + bias) in float32 (or, with `softmax`, the softmax of router h + bias over all entries; `normalize` then makes it the
+    softmax over the chosen ones), choice by score + correction, chosen
     scores over their sum (+ 1e-20) if `normalize`, times scale. The router's rows: the experts, then `identity` entries
     that are chosen like experts but have no weights (the sum of a row's chosen identity weights leaves in the LAST column
     of `weights`), then `gates` rows that are not routed: sigmoid(row . h) * scale leaves in the columns behind the experts'.
@@ -470,7 +503,9 @@ def route_experts(h, router, correction, top, scale, normalize, weights, identit
     assert router.dtype == torch.float32 and router.is_contiguous() and weights.dtype == torch.float32
     real = router.shape[0] - identity - gates
     assert weights.is_contiguous() and h.stride(1) == 1 and weights.shape == (h.shape[0], real + gates + (1 if identity else 0))
-    _call("jllm_route_experts", h.data_ptr(), _DT[h.dtype], h.stride(0), router.data_ptr(), _p(correction),
+    assert bias is None or (bias.is_contiguous() and bias.numel() == real + identity)
+    _call("jllm_route_experts", h.data_ptr(), _DT[h.dtype], h.stride(0), router.data_ptr(), _p(bias),
+          _DT[bias.dtype] if bias is not None else F32, _p(correction),
           _DT[correction.dtype] if correction is not None else F32, weights.data_ptr(), h.shape[0], h.shape[1],
           real, int(top), float(scale), int(bool(normalize)), int(identity), int(gates), int(bool(softmax)), weights.shape[1],
           _stream())
@@ -620,9 +655,32 @@ def glu_descriptor(activation: str, limit: float = 0.0) -> int:
     return (bits & ~3) | 3
 
 
+class _GluMore(ctypes.Structure):          # (GluMore in common.cuh)
+    _fields_ = [("word_behind", c_int), ("split", c_int), ("ff", c_int), ("ld_w", c_int), ("weights", c_void_p)]
+
+
+class GluUnits:
+    """A product's `swiglu` argument where the stacked units are several feed-forwards': units from `split` on (0: none) have an
+    activation word of their own, and with `weights` ([rows, columns] float32) unit u's result is multiplied by weights[row, u // ff],
+    a unit's from `split` on by weights[row, split // ff]."""
+
+    def __init__(self, word: int, ff: int, split: int = 0, word_behind: int = 0, weights: torch.Tensor | None = None):
+        assert weights is None or (weights.dtype == torch.float32 and weights.stride(1) == 1)
+        self.word, self.weights = int(word), weights
+        self._more = _GluMore(int(word_behind), int(split), int(ff), weights.stride(0) if weights is not None else 0, _p(weights))
+        self.more = ctypes.addressof(self._more)
+
+
+def glu_more(activation) -> int:
+    """The address of what a product is told beyond the activation's word, or 0."""
+    return activation.more if isinstance(activation, GluUnits) else 0
+
+
 def glu_kind(activation) -> int:
     """0 (no gating), or the kernels' number of a gated feed-forward's activation; True stands for silu. The products take
     it as their `swiglu` argument: False, True, or the activation's name."""
+    if isinstance(activation, GluUnits):
+        return activation.word
     if isinstance(activation, (bool, int)):
         return int(activation)
     return GLU_KINDS[activation] if activation else 0
@@ -650,17 +708,19 @@ def head_prepare(qkv, q_off, k_off, v_off, q_gain, k_gain, eps, cos, sin, rotary
 
 
 def map_prepare(src, k_off, v_off, q_gain, k_gain, eps, cos, sin, rotary_dim, pairing, positions, slots, q_out, k_cache, v_cache,
-                heads, kv_heads, maps, dim, value_dim, width, page_size, write_kv=True) -> None:
+                heads, kv_heads, maps, dim, value_dim, width, page_size, write_kv=True, temp_every: int = 0,
+                temp_coef: float = 0.0) -> None:
     """The rows of a wide attention (see attention_maps.cu) from the stacked projection `src` [rows, *] (queries at column 0): an
     optional RMS norm over all query (key) columns of a row with float32 gains per column; the rotation of the first `rotary_dim`
     values of every map; query (head, map) to its own `width` values of q_out with zeros around it, the maps of a key head side by
-    side into one cache row, the value into another, zeros behind both. `write_kv` False: queries only."""
+    side into one cache row, the value into another, zeros behind both. `write_kv` False: queries only. v_off = k_off: the values
+    are the keys as projected. `temp_every` > 0: queries times 1 + temp_coef ln(floor((position + 1) / temp_every) + 1)."""
     assert src.stride(1) == 1 and q_out.dtype == src.dtype and q_out.stride(1) == 1
     assert all(g is None or (g.dtype == torch.float32 and g.is_contiguous()) for g in (q_gain, k_gain))
     _call("jllm_map_prepare", src.data_ptr(), _DT[src.dtype], src.stride(0), int(k_off), int(v_off), _p(q_gain), _p(k_gain),
           float(eps), _p(cos), _p(sin), int(rotary_dim), {"half": 0, "interleaved": 1}[pairing], positions.data_ptr(), _p(slots),
           q_out.data_ptr(), q_out.stride(0), _p(k_cache), _p(v_cache), int(write_kv), src.shape[0], heads, kv_heads, maps, dim,
-          value_dim, width, page_size, _stream())
+          value_dim, width, page_size, int(temp_every), float(temp_coef), _stream())
 
 
 def map_difference(att, width, lam, eps, out_scale, out, heads, value_dim) -> None:
@@ -785,15 +845,17 @@ def norm_chain(x, a, gain_post, eps, b=None, gain_a=None, gain_b=None, scale: fl
 
 
 def attention_plain(q, q_stride, k_cache, v_cache, out, row_seg, row_pos, block_tables, rows, heads, kv_heads,
-                    head_dim, page_size, window, scale, value_dim: int = 0, keep_first: int = 0, sink=None) -> None:
+                    head_dim, page_size, window, scale, value_dim: int = 0, keep_first: int = 0, sink=None,
+                    softcap: float = 0.0) -> None:
     """`window`: 0 all earlier keys, w > 0 the last w keys, -c < 0 the keys of the row's own chunk of c positions.
     `keep_first` (with a window): the request's first keys stay visible. `sink` [heads]: exp(sink) joins the denominator.
+    `softcap` > 0: a score s = scale (q . k) becomes softcap * tanh(s / softcap).
     `value_dim` (0: head_dim): the width of a value head where it differs from a key head's; the cache's rows are as
     wide as k_cache's last dimension says."""
     _call("jllm_attention_plain", q.data_ptr(), q_stride, k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
           out.stride(0), row_seg.data_ptr(), row_pos.data_ptr(), block_tables.data_ptr(), block_tables.stride(0),
           rows, heads, kv_heads, head_dim, int(value_dim or head_dim), k_cache.shape[-1], page_size, int(window),
-          float(scale), _DT[q.dtype], int(keep_first), _p(sink), _DT[sink.dtype] if sink is not None else F32, _stream())
+          float(scale), _DT[q.dtype], int(keep_first), _p(sink), _DT[sink.dtype] if sink is not None else F32, float(softcap), _stream())
 
 
 def argmax(logits: torch.Tensor, out: torch.Tensor, vocab: int | None = None) -> None:
@@ -936,7 +998,7 @@ def gemm_tcgen05(a, w, out, bias=None, accumulate=False, max_blocks: int = 0, sw
     ws = gemm_workspace(a.device, STREAM_WORKSPACE_FLOATS) if stream_mode == 1 else None
     _call("jllm_gemm_tcgen05", a.data_ptr(), a.stride(0), w.data.data_ptr(), w.k_blocks, _p(bias),
           _DT[bias.dtype] if bias is not None else F32, out.data_ptr(), _DT[out.dtype], out.stride(0),
-          int(accumulate), a.shape[0], w.rows, w.cols, int(max_blocks), glu_kind(swiglu), _p(ws),
+          int(accumulate), a.shape[0], w.rows, w.cols, int(max_blocks), glu_kind(swiglu), glu_more(swiglu), _p(ws),
           ws.numel() if ws is not None else 0, int(stream_mode), int(tile_width), _stream())
 
 
@@ -950,7 +1012,7 @@ def gemm_pair(a, w, out, bias=None, accumulate=False, swiglu=False, max_pairs: i
     ws = gemm_workspace((a.device, "pair"), PAIR_WORKSPACE_FLOATS) if stream_mode == 1 else None
     _call("jllm_gemm_pair", a.data_ptr(), a.stride(0), w.data.data_ptr(), w.k_blocks, _p(bias),
           _DT[bias.dtype] if bias is not None else F32, out.data_ptr(), _DT[out.dtype], out.stride(0),
-          int(accumulate), a.shape[0], w.rows, w.cols, int(max_pairs), glu_kind(swiglu), _p(ws),
+          int(accumulate), a.shape[0], w.rows, w.cols, int(max_pairs), glu_kind(swiglu), glu_more(swiglu), _p(ws),
           ws.numel() if ws is not None else 0, int(stream_mode), _stream())
 
 
@@ -1030,7 +1092,7 @@ def gemm_stream(a, packed: PackedWeight, out, bias=None, accumulate=False, swigl
     ws = gemm_workspace((a.device, "stream"), SWAP_WORKSPACE_FLOATS)     # its own: it keeps counters of its own there
     _call("jllm_gemm_stream", a.data_ptr(), a.stride(0), packed.data.data_ptr(), packed.k_blocks, _p(bias),
           _DT[bias.dtype] if bias is not None else F32, out.data_ptr(), _DT[out.dtype], out.stride(0), int(accumulate),
-          a.shape[0], packed.rows, packed.cols, glu_kind(swiglu), ws.data_ptr(), ws.numel(), int(max_blocks), _stream())
+          a.shape[0], packed.rows, packed.cols, glu_kind(swiglu), glu_more(swiglu), ws.data_ptr(), ws.numel(), int(max_blocks), _stream())
 
 
 BOUNDS_FILES = ("attention_plain", "attention_decode", "attention_prefill", "attention_prefill_tc",
@@ -1111,7 +1173,7 @@ def gemm_small_m(a, w, out, bias=None, accumulate=False, swiglu=False) -> None:
     assert a.dtype == torch.bfloat16 and out.stride(-1) == 1 and a.shape[1] == w.cols
     _call("jllm_gemm_small_m", a.data_ptr(), a.stride(0), w.data.data_ptr(), w.k_blocks, _p(bias),
           _DT[bias.dtype] if bias is not None else F32, out.data_ptr(), _DT[out.dtype], out.stride(0),
-          int(accumulate), a.shape[0], w.rows, w.cols, glu_kind(swiglu), _stream())
+          int(accumulate), a.shape[0], w.rows, w.cols, glu_kind(swiglu), glu_more(swiglu), _stream())
 
 
 def attention_decode_fits(dtype, heads, kv_heads, head_dim) -> bool:
@@ -1140,7 +1202,7 @@ def attention_decode_flat_scratch_floats(rows, heads, kv_heads, head_dim, blocks
 
 
 def attention_decode_flat(q, k_cache, v_cache, out, row_seg, row_pos, block_tables, rows, heads, kv_heads, head_dim,
-                          page_size, window, scale, blocks, scratch) -> None:
+                          page_size, window, scale, blocks, scratch, softcap: float = 0.0) -> None:
     """One query position per row, the key tiles of all (row, kv head) pairs dealt out evenly over `blocks` blocks."""
     assert scratch.dtype == torch.float32 and \
         scratch.numel() >= attention_decode_flat_scratch_floats(rows, heads, kv_heads, head_dim, blocks)
@@ -1148,7 +1210,8 @@ def attention_decode_flat(q, k_cache, v_cache, out, row_seg, row_pos, block_tabl
     launch_count += _combine_launches("flat", blocks, rows, kv_heads, head_dim)
     _call("jllm_attention_decode_flat", q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
           out.stride(0), row_seg.data_ptr(), row_pos.data_ptr(), block_tables.data_ptr(), block_tables.stride(0),
-          rows, heads, kv_heads, head_dim, page_size, int(window), float(scale), int(blocks), scratch.data_ptr(), _stream())
+          rows, heads, kv_heads, head_dim, page_size, int(window), float(scale), int(blocks), scratch.data_ptr(), float(softcap),
+          _stream())
 
 
 FLAT_DECODE = int(os.environ.get("JLLM_B200_FLAT_DECODE", "1"))
@@ -1203,32 +1266,36 @@ def decode_bucket_cap(rows, kv_heads, heads, head_dim, window, scratch, places: 
 
 
 def attention_decode_extras(q, k_cache, v_cache, out, row_seg, row_pos, block_tables, rows, heads, kv_heads, head_dim,
-                            page_size, window, scale, splits=1, scratch=None, keep_first: int = 0, sink=None) -> None:
+                            page_size, window, scale, splits=1, scratch=None, keep_first: int = 0, sink=None,
+                            softcap: float = 0.0) -> None:
     """`attention_decode` with a window that keeps the request's first `keep_first` keys visible and / or a sink per query
-    head: the general kernel for every head size (a row's visible keys are walked by an index that counts them), the sink
+    head and / or a cap on the scores (`softcap` > 0: s becomes softcap * tanh(s / softcap)): the general kernel for every head size (a row's visible keys are walked by an index that counts them), the sink
     added where a row's parts meet."""
     if splits > 1:
         assert scratch is not None and scratch.dtype == torch.float32 and \
             scratch.numel() >= attention_decode_scratch_floats(rows, heads, head_dim, splits)
     global launch_count
-    launch_count += 1 if splits > 1 else 0
+    launch_count += _combine_launches("split", splits, rows, kv_heads, head_dim)
     _call("jllm_attention_decode_extras", q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
           out.stride(0), row_seg.data_ptr(), row_pos.data_ptr(), block_tables.data_ptr(), block_tables.stride(0),
           rows, heads, kv_heads, head_dim, page_size, int(window), float(scale), int(splits), _p(scratch), int(keep_first),
-          _p(sink), _DT[sink.dtype] if sink is not None else F32, _stream())
+          _p(sink), _DT[sink.dtype] if sink is not None else F32, float(softcap), _stream())
 
 
 def _attention_decode_rows(q, k_cache, v_cache, out, row_seg, positions, table, rows, heads, kv_heads, head_dim, page_size,
-                           window, scale, kv_bucket, scratch, keep_first: int = 0, sink=None):
+                           window, scale, kv_bucket, scratch, keep_first: int = 0, sink=None, softcap: float = 0.0):
     bucket = _windowed_bucket(kv_bucket, window)
     if keep_first or sink is not None:
         splits = decode_splits(rows, kv_heads, bucket, heads, head_dim, scratch)
         return attention_decode_extras(q, k_cache, v_cache, out, row_seg, positions, table, rows, heads, kv_heads, head_dim,
-                                       page_size, window, scale, splits, scratch, keep_first, sink)
+                                       page_size, window, scale, splits, scratch, keep_first, sink, softcap)
     how, n = decode_plan(rows, kv_heads, bucket, heads, head_dim, scratch)
     if how == "flat":
         return attention_decode_flat(q, k_cache, v_cache, out, row_seg, positions, table, rows, heads, kv_heads, head_dim,
-                                     page_size, window, scale, n, scratch)
+                                     page_size, window, scale, n, scratch, softcap)
+    if softcap:
+        return attention_decode_extras(q, k_cache, v_cache, out, row_seg, positions, table, rows, heads, kv_heads, head_dim,
+                                       page_size, window, scale, n, scratch, 0, None, softcap)
     return attention_decode(q, k_cache, v_cache, out, row_seg, positions, table, rows, heads, kv_heads, head_dim, page_size,
                             window, scale, n, scratch)
 
@@ -1277,20 +1344,20 @@ def _combine_launches(how, n, rows, kv_heads, head_dim) -> int:
 
 
 def attention(q, k_cache, v_cache, out, batch, group, heads, kv_heads, head_dim, page_size, window, scale,
-              scratch=None, value_dim: int = 0, keep_first: int = 0, sink=None) -> None:
+              scratch=None, value_dim: int = 0, keep_first: int = 0, sink=None, softcap: float = 0.0) -> None:
     """Causal attention of every row of the batch over its own request's cached keys and values. `window`: 0 every
     earlier key, w > 0 the last w keys, -c < 0 the keys of the row's own chunk of c positions (position p lies in chunk
     p // c). `value_dim`: a value head's width where it is not `head_dim`; the tile kernels take heads
     of one width only, so such a mixer runs on the plain kernel. `keep_first` (with a window): the request's first keys stay
-    visible to every row. `sink` [heads]: a number per query head whose exponential joins the softmax's denominator. With
-    either, single rows run on the general decode kernel and prompt portions on the tcgen05 kernel of one query tile (heads of
+    visible to every row. `sink` [heads]: a number per query head whose exponential joins the softmax's denominator. `softcap`
+    > 0: every score s = scale (q . k) becomes softcap * tanh(s / softcap), in every kernel. With kept keys or a sink, single rows run on the general decode kernel and prompt portions on the tcgen05 kernel of one query tile (heads of
     128) or the mma.sync kernel (64, 256)."""
     one_width = value_dim in (0, head_dim) and k_cache.shape[-1] == head_dim
     extras = bool(keep_first) or sink is not None
     if one_width and batch.decode_only and attention_decode_fits(q.dtype, heads, kv_heads, head_dim):
         return _attention_decode_rows(q, k_cache, v_cache, out, batch.row_seg, batch.positions, batch.block_tables[group],
                                       batch.rows, heads, kv_heads, head_dim, page_size, window, scale, batch.kv_bucket,
-                                      scratch, keep_first, sink)
+                                      scratch, keep_first, sink, softcap)
     if one_width and q.dtype == torch.bfloat16 and attention_prefill_fits(head_dim):
         # prompt portions through the flash kernel; the single rows riding beside them (the scheduler puts them
         # last) through the decode kernel, which shares every key among the query heads of a kv head
@@ -1300,15 +1367,15 @@ def attention(q, k_cache, v_cache, out, batch, group, heads, kv_heads, head_dim,
         if mr > 0:
             attention_prefill(q[:mr], k_cache, v_cache, out[:mr], batch.seg_start[:ms], batch.seg_len[:ms],
                               batch.seg_kv_len[:ms], batch.block_tables[group], mr, heads, kv_heads, head_dim, page_size,
-                              window, scale, keep_first=keep_first, sink=sink)
+                              window, scale, keep_first=keep_first, sink=sink, softcap=softcap)
         if mr < batch.rows:
             n = batch.rows - mr
             _attention_decode_rows(q[mr:], k_cache, v_cache, out[mr:], batch.row_seg[mr:], batch.positions[mr:],
                                    batch.block_tables[group], n, heads, kv_heads, head_dim, page_size, window, scale,
-                                   batch.kv_bucket, scratch, keep_first, sink)
+                                   batch.kv_bucket, scratch, keep_first, sink, softcap)
         return
     attention_plain(q, q.stride(0), k_cache, v_cache, out, batch.row_seg, batch.positions, batch.block_tables[group],
-                    batch.rows, heads, kv_heads, head_dim, page_size, window, scale, value_dim, keep_first, sink)
+                    batch.rows, heads, kv_heads, head_dim, page_size, window, scale, value_dim, keep_first, sink, softcap)
 
 
 def attention_tiles_take(keep_first: int, sink) -> bool:
@@ -1330,7 +1397,8 @@ def attention_prefill_tc_fits(q, out, k_cache, head_dim, page_size) -> bool:
 
 
 def attention_prefill(q, k_cache, v_cache, out, seg_start, seg_len, seg_kv_len, block_tables, rows, heads, kv_heads,
-                      head_dim, page_size, window, scale, kernel: str = "auto", keep_first: int = 0, sink=None) -> None:
+                      head_dim, page_size, window, scale, kernel: str = "auto", keep_first: int = 0, sink=None,
+                      softcap: float = 0.0) -> None:
     """Flash attention of prompt portions: segments of consecutive rows, each over its own request's pages.
     Head size 128 runs on tcgen05 (both products, accumulators in tensor memory; kernel "pair" or "tc"), other
     sizes on mma.sync ("mma")."""
@@ -1338,7 +1406,7 @@ def attention_prefill(q, k_cache, v_cache, out, seg_start, seg_len, seg_kv_len, 
         # two query tiles per block where the portions are long enough to fill them (the tiles take turns on the
         # tensor cores); one tile per block, with two S buffers, for short portions
         kernel = "pair" if rows > 128 * seg_start.numel() and PREFILL_TC != 3 else "tc"
-    if keep_first or sink is not None:
+    if keep_first or sink is not None or (softcap and kernel != "pair"):
         # kept first keys and a sink: the tcgen05 kernel of one query tile per block, or the mma.sync kernel
         kernel = "tc" if kernel in ("tc", "pair") else "mma"
         sd = _DT[sink.dtype] if sink is not None else F32
@@ -1346,16 +1414,18 @@ def attention_prefill(q, k_cache, v_cache, out, seg_start, seg_len, seg_kv_len, 
             return _call("jllm_attention_prefill_tc_extras", q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
                          k_cache.shape[0], out.data_ptr(), out.stride(0), seg_start.data_ptr(), seg_len.data_ptr(),
                          seg_kv_len.data_ptr(), block_tables.data_ptr(), block_tables.stride(0), seg_start.numel(), rows,
-                         heads, kv_heads, head_dim, page_size, int(window), float(scale), int(keep_first), _p(sink), sd, _stream())
+                         heads, kv_heads, head_dim, page_size, int(window), float(scale), int(keep_first), _p(sink), sd, float(softcap),
+                         _stream())
         return _call("jllm_attention_prefill_extras", q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
                      out.data_ptr(), out.stride(0), seg_start.data_ptr(), seg_len.data_ptr(), seg_kv_len.data_ptr(),
                      block_tables.data_ptr(), block_tables.stride(0), seg_start.numel(), rows, heads, kv_heads, head_dim,
-                     page_size, int(window), float(scale), int(keep_first), _p(sink), sd, _stream())
+                     page_size, int(window), float(scale), int(keep_first), _p(sink), sd, float(softcap), _stream())
     if kernel in ("tc", "pair"):
         return _call("jllm_attention_prefill_tc" if kernel == "tc" else "jllm_attention_prefill_pair", q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
                      k_cache.shape[0], out.data_ptr(), out.stride(0), seg_start.data_ptr(), seg_len.data_ptr(),
                      seg_kv_len.data_ptr(), block_tables.data_ptr(), block_tables.stride(0), seg_start.numel(), rows,
-                     heads, kv_heads, head_dim, page_size, int(window), float(scale), _stream())
+                     heads, kv_heads, head_dim, page_size, int(window), float(scale),
+                     *((float(softcap),) if kernel == "pair" else ()), _stream())
     _call("jllm_attention_prefill", q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
           out.stride(0), seg_start.data_ptr(), seg_len.data_ptr(), seg_kv_len.data_ptr(), block_tables.data_ptr(),
           block_tables.stride(0), seg_start.numel(), rows, heads, kv_heads, head_dim, page_size, int(window),

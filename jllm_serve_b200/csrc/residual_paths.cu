@@ -15,6 +15,7 @@
 //                    block per row: x[r] += norm(a[r]) * w is the newest plane of the stack, the mix of all planes goes to the
 //                    plane behind it, and its blend with the next layer's saved row leaves in the compute type
 //   scale_values     x *= s
+//   softcap_values   x = c tanh(x / c)
 //
 // and in front of a part whose input is blended over time:
 //   norm_conv        h = rms(x) * w;  out[r] = h_t + sum_j c[:, j] h_(t - taps + 1 + j) per channel: the layer's norm and a short
@@ -276,6 +277,13 @@ __global__ void scale_values_kernel(float* __restrict__ x, float s, size_t count
     pdl_trigger();
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < count; i += (size_t)gridDim.x * blockDim.x)
         x[i] = __fmul_rn(x[i], s);
+}
+
+__global__ void softcap_values_kernel(float* __restrict__ x, float cap, size_t count) {
+    pdl_wait();
+    pdl_trigger();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < count; i += (size_t)gridDim.x * blockDim.x)
+        x[i] = __fmul_rn(cap, tanhf(x[i] / cap));
 }
 
 // The rms factors of the rows [lo, hi) into `inv` (a warp per row).
@@ -560,6 +568,14 @@ JLLM_EXPORT int jllm_scale_values(float* x, float s, long long count, cudaStream
     const int blocks = (int)min((size_t)65535, ((size_t)count + 255) / 256);
     jllm_launch(scale_values_kernel, dim3(blocks), dim3(256), 0, stream, LAUNCH_DEPENDENT, x, s, (size_t)count);
     return jllm_check_launch("scale_values");
+}
+
+JLLM_EXPORT int jllm_softcap_values(float* x, float cap, long long count, cudaStream_t stream) {
+    JLLM_REQUIRE(count >= 0, "softcap_values: count=%lld", count);
+    if (count == 0) return JLLM_OK;
+    const int blocks = (int)min((size_t)65535, ((size_t)count + 255) / 256);
+    jllm_launch(softcap_values_kernel, dim3(blocks), dim3(256), 0, stream, LAUNCH_DEPENDENT, x, cap, (size_t)count);
+    return jllm_check_launch("softcap_values");
 }
 
 // x [rows, dim] float32; gain [dim] and conv [dim, taps] of types `gain_dtype` and `conv_dtype`; state [slots, max(taps - 1, 1), dim]

@@ -53,6 +53,10 @@ class DecoderModel:
         self.vocab, self.dim = core.vocab, core.dim
         self.logit_scale = float(getattr(core, "logit_scale", 1.0))
         self.embedding_scale = float(getattr(core, "embedding_scale", 1.0))
+        self.logit_softcap = float(getattr(core, "logit_softcap", 0.0))
+        self.streams = int(getattr(core, "streams", 0))
+        if self.streams:
+            self._all_streams = torch.ones(self.streams, dtype=torch.float32, device=runtime.device)
         # depth mix: what run i hands on is a weighted sum of the embedded rows and of every run's result so far
         self.depth_weights = None
         if getattr(spec, "depth_mix", ""):
@@ -139,6 +143,19 @@ class DecoderModel:
             out.block_states = tuple(cache.states(i)[-mine:])
         return out
 
+    def _run_streams(self, x, batch, cache, n: int, head_in) -> None:
+        """The layer runs over a residual of several streams; leaves the head's input for the batch's `n` wanted rows in `head_in`."""
+        schedule = self.spec.schedule
+        streams = self.rt.buffer("streams", self.streams * self.dim, torch.float32)[:batch.rows].view(-1, self.streams, self.dim)
+        xb = self.rt.buffer("normed", self.dim)[:batch.rows]
+        norm = self.final_norm
+        for i, run in enumerate(schedule):
+            if i + 1 < len(schedule):
+                tail = (*self.blocks[schedule[i + 1].layer].opening(), xb, None)
+            else:          # the sum of the streams and the last norm, for the rows that are asked for
+                tail = (self._all_streams, norm.gain, norm.eps, head_in, batch.logit_rows) if n else None
+            self.blocks[run.layer].forward(streams, batch, self._run_cache(cache, i), start=x if i == 0 else None, tail=tail)
+
     def forward(self, batch, cache, logits_out: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Runs the batch's rows through every scheduled layer; returns float32 logits [wanted rows, vocab]."""
         rows = batch.rows
@@ -156,6 +173,11 @@ class DecoderModel:
         ops.embed_rows(batch.token_ids, self.embedding, x, self.embedding_scale)
         for pe in self.position_encodings:
             pe.on_embedding(x, batch)
+        if self.streams:
+            n = batch.num_wanted
+            hb = self.rt.buffer("head_in", self.dim)[:n]
+            self._run_streams(x, batch, cache, n, hb)
+            return self._logits(hb, n, logits_out)
         for i, run in enumerate(schedule):
             block = self.blocks[run.layer]
             if stack is not None:
@@ -185,15 +207,22 @@ class DecoderModel:
                 ops.depth_mix(stack, self.depth_weights[i], i + 2, stack[i + 2])
                 x = stack[i + 2]
         n = batch.num_wanted
+        hb = self.rt.buffer("head_in", self.dim)[:n]
+        if n:
+            self.final_norm.forward(x, hb, row_index=batch.logit_rows, rows=n)
+        return self._logits(hb, n, logits_out)
+
+    def _logits(self, hb, n: int, logits_out) -> torch.Tensor:
+        """The head's product for `n` normed rows, and what the model does to its result."""
         if logits_out is None:
             logits_out = torch.empty((n, self.vocab), dtype=torch.float32, device=self.rt.device)
         if n == 0:
             return logits_out[:0]
-        hb = self.rt.buffer("head_in", self.dim)[:n]
-        self.final_norm.forward(x, hb, row_index=batch.logit_rows, rows=n)
         self.head.forward(hb, logits_out[:n])
         if self.logit_scale != 1.0:
             ops.scale_values(logits_out[:n], self.logit_scale)
+        if self.logit_softcap:
+            ops.softcap_values(logits_out[:n], self.logit_softcap)
         return logits_out[:n]
 
 

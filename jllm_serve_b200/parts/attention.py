@@ -28,7 +28,9 @@ copy of the values: a cached key row holds [map 1, map 2], a query head becomes 
 attention kernels see heads x 2 query heads over kv_heads plain heads; `ops.map_difference` then subtracts the second map's
 result (times lambda, a number of the layer made from four stored vectors), norms the difference per head and scales it. Rows are
 filled up with zeros to a width the tile kernels take where that costs little (`spec.row_dim`). With `own_kv` False there are no
-key and value projections: the run reads what another run cached, under its own mask.
+key and value projections: the run reads what another run cached, under its own mask. The same preparation multiplies queries that
+grow with their position (`temp_every`) and, with `keys_as_values`, caches the keys' raw columns as the values (one projection). A cap
+on the scores (`softcap`) is the attention kernels' own, in every form.
 """
 from __future__ import annotations
 
@@ -107,13 +109,18 @@ class GqaAttention(Mixer):
         self.k_off, self.v_off, self.width = 0, 0, q_width
         if s.own_kv:
             rows, at = [], 0
-            for t, n in ((w[0], q_width), (tensors.pop(prefix + names.k), k_width), (tensors.pop(prefix + names.v), v_width)):
+            pieces = [(w[0], q_width), (tensors.pop(prefix + names.k), k_width)]
+            if not s.keys_as_values:
+                pieces.append((tensors.pop(prefix + names.v), v_width))
+            for t, n in pieces:
                 if at != _up8(at):       # every piece starts at a multiple of 8 columns
                     rows.append(torch.zeros((_up8(at) - at, self.dim), dtype=t.dtype, device=t.device))
                     at = _up8(at)
                 rows.append(t)
                 self.k_off, self.v_off = self.v_off, at
                 at += n
+            if s.keys_as_values:
+                self.k_off = self.v_off
             w, self.width = rows, at
         self.qkv = Linear(torch.cat(w, dim=0).contiguous())
         del w
@@ -146,7 +153,9 @@ class GqaAttention(Mixer):
         q_width, k_width = s.heads * s.maps * s.head_dim, s.kv_heads * s.maps * s.head_dim
         out = {prefix + names.q: TensorWant((q_width, dim)), prefix + names.o: TensorWant((dim, s.heads * s.v_dim))}
         if s.own_kv:
-            out.update({prefix + names.k: TensorWant((k_width, dim)), prefix + names.v: TensorWant((s.kv_heads * s.v_dim, dim))})
+            out[prefix + names.k] = TensorWant((k_width, dim))
+            if not s.keys_as_values:
+                out[prefix + names.v] = TensorWant((s.kv_heads * s.v_dim, dim))
         if s.qk_norm:
             out[prefix + names.q_norm] = TensorWant((q_width,), "vector", init="gain")
             if s.own_kv:
@@ -216,11 +225,12 @@ class GqaAttention(Mixer):
         ops.map_prepare(qkv, self.k_off, self.v_off, self.q_gain, self.k_gain, s.qk_norm_eps, rope.cos if rope else None,
                         rope.sin if rope else None, rope.rotary_dim if rope else 0, rope.pairing if rope else "half",
                         batch.positions, batch.slots[cache.group] if cache.writes else None, q, cache.keys, cache.values, s.heads,
-                        s.kv_heads, s.maps, s.head_dim, s.v_dim, W, self.rt.page_size, write_kv=cache.writes)
+                        s.kv_heads, s.maps, s.head_dim, s.v_dim, W, self.rt.page_size, write_kv=cache.writes,
+                        temp_every=s.temp_every, temp_coef=s.temp_coef)
         att = self.rt.buffer("attention_out", heads * W)[:rows]
         scratch = self.rt.buffer("attention_scratch", 2 << 20, torch.float32, rows=1)[0]
         ops.attention(q, cache.keys, cache.values, att, batch, cache.group, heads, s.kv_heads, W, self.rt.page_size, self.span,
-                      s.scale, scratch, keep_first=self.keep_first)
+                      s.scale, scratch, keep_first=self.keep_first, softcap=s.softcap)
         if s.maps == 2:
             y = self.rt.buffer("map_difference", s.heads * s.v_dim)[:rows]
             ops.map_difference(att, W, self.lam, s.diff_norm_eps, 1.0 - s.diff, y, s.heads, s.v_dim)
@@ -243,7 +253,7 @@ class GqaAttention(Mixer):
         att = self.rt.buffer("attention_out", s.heads * s.v_dim)[:rows]
         scratch = self.rt.buffer("attention_scratch", 2 << 20, torch.float32, rows=1)[0]
         if (self.classic and not self.gated and cache.writes and batch.decode_only and rope is not None
-                and self.sink is None and not self.keep_first and self.out_scale == 1.0
+                and self.sink is None and not self.keep_first and self.out_scale == 1.0 and not s.softcap
                 and ops.attention_decode_fits(qkv.dtype, s.heads, s.kv_heads, s.head_dim)
                 and ops.attention_decode_fresh_fits(qkv.dtype, s.heads, s.kv_heads, s.head_dim, rope.rotary_dim)):
             # a step of single rows: the attention kernel norms and rotates its own rows and writes their keys and values
@@ -266,7 +276,7 @@ class GqaAttention(Mixer):
                              s.heads, s.kv_heads, s.head_dim, s.v_dim, self.rt.page_size, write_kv=cache.writes)
         ops.attention(qkv, cache.keys, cache.values, att, batch, cache.group, s.heads, s.kv_heads, s.head_dim,
                       self.rt.page_size, self.span, s.scale, scratch, value_dim=s.v_dim, keep_first=self.keep_first,
-                      sink=self.sink)
+                      sink=self.sink, softcap=s.softcap)
         if s.gate == "sigmoid":
             ops.sigmoid_gate(att, qkv[:, self.g_off:self.g_off + self.gate_width], self.out_scale)
         else:

@@ -338,3 +338,108 @@ class PostNormBlock(Block):
 
 
 register_block("post_norm", PostNormBlock, replace=True)
+
+
+class HyperConnectionBlock(Block):
+    """A residual of several streams X_1 .. X_S in place of one (float32, [rows, S, dim]; all begin as the embedded rows):
+
+        u = sum_s in[s] X_s;   y = part(norm(u));   X_t <- sum_s mix[s, t] X_s + out[t] y
+
+    for the mixer (`names.mixer_streams`) and the feed-forward (`names.feed_forward_streams`), each with vectors and a matrix of its
+    own. A part writes its result into a float32 buffer (`overwrite`; one that cannot gets it zeroed); one launch then mixes the
+    streams and makes the normed input of the part that follows: the feed-forward's, or the next block's mixer's, or, behind the
+    last block, the head's for the rows that are asked for (`ops.stream_mix`; the model hands a block what follows it as `tail`)."""
+
+    streams_residual = True      # `forward` takes the streams, `start` and `tail`
+
+    def __init__(self, spec, dim: int, tensors: dict, prefix: str, runtime, position_encodings):
+        names, gain = spec.names, getattr(spec.norm, "gain_name", "weight")
+        if spec.norm.kind != "rmsnorm" or spec.streams < 1 or float(getattr(spec, "residual_scale", 1.0)) != 1.0:
+            raise ValueError("hyper-connections: one or more streams, RMS norms and no residual scale")
+        self.rt, self.dim, self.eps, self.streams = runtime, dim, float(spec.norm.eps), spec.streams
+        self.mixer_gain = tensors[prefix + names.mixer_norm + gain]
+        mixer_cls = part_class("mixer", spec.mixer.kind)
+        table = getattr(spec.mixer, "rope_table", -1)
+        extra = {"rope": position_encodings[table]} if table is not None and table >= 0 and position_encodings else {}
+        if getattr(mixer_cls, "wants_position_encodings", False):
+            extra = {"position_encodings": position_encodings}
+        self.mixer = mixer_cls(spec.mixer, dim, tensors, prefix + names.mixer, runtime, **extra)
+        self.mixer_read, self.mixer_mix = self._weights(tensors, prefix + names.mixer_streams)
+        self.ffn_gain = self.feed_forward = None
+        if spec.feed_forward is not None:
+            self.ffn_gain = tensors[prefix + names.feed_forward_norm + gain]
+            self.feed_forward = part_class("feed_forward", spec.feed_forward.kind)(
+                spec.feed_forward, dim, tensors, prefix + names.feed_forward, runtime)
+            self.ffn_read, self.ffn_mix = self._weights(tensors, prefix + names.feed_forward_streams)
+        self._zero_first = set()
+        for part in (self.mixer, self.feed_forward):
+            if part is None:
+                continue
+            if getattr(part, "can_overwrite", False):
+                part.overwrite = True
+            else:
+                self._zero_first.add(id(part))
+
+    def _weights(self, tensors: dict, name: str):
+        """(in [S], mix [S, S] with out [S] behind it), float32: how the kernel takes them."""
+        read, mix, out = (tensors[name + n].float() for n in ("in", "mix", "out"))
+        return read.contiguous(), torch.cat([mix.reshape(-1), out]).contiguous()
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(getattr(p, "graph_safe", False) for p in (self.mixer, self.feed_forward) if p is not None)
+
+    def decode_bucket_cap(self, rows: int) -> int:
+        return getattr(self.mixer, "decode_bucket_cap", lambda _: 32)(rows)
+
+    @classmethod
+    def wants(cls, spec, dim: int, prefix: str) -> dict:
+        names, gain, S = spec.names, getattr(spec.norm, "gain_name", "weight"), spec.streams
+
+        def streams(name):
+            return {name + "in": TensorWant((S,), "vector", init="average"), name + "out": TensorWant((S,), "vector", init="gain"),
+                    name + "mix": TensorWant((S, S), "vector", init="identity")}
+        out = {prefix + names.mixer_norm + gain: TensorWant((dim,), "vector", init="gain")}
+        out.update(part_class("mixer", spec.mixer.kind).wants(spec.mixer, dim, prefix + names.mixer))
+        out.update(streams(prefix + names.mixer_streams))
+        if spec.feed_forward is not None:
+            out[prefix + names.feed_forward_norm + gain] = TensorWant((dim,), "vector", init="gain")
+            out.update(part_class("feed_forward", spec.feed_forward.kind).wants(spec.feed_forward, dim,
+                                                                                prefix + names.feed_forward))
+            out.update(streams(prefix + names.feed_forward_streams))
+        return out
+
+    def _result(self, part, rows):
+        y = self.rt.buffer("part_result", self.dim, torch.float32)[:rows]
+        if id(part) in self._zero_first:
+            y.zero_()
+        return y
+
+    def opening(self) -> tuple:
+        """(in, gain, eps): what makes this block's first input out of the streams."""
+        return self.mixer_read, self.mixer_gain, self.eps
+
+    def forward(self, streams, batch, cache, start=None, tail=None) -> None:
+        """`start`: the embedded rows, for the first block (the streams are made from them; else the block in front has left this
+        block's input in the shared buffer of normed rows). `tail`: (in, gain, eps, out, rows or None) of what follows: its normed
+        input goes to `out`, and with `rows` only those rows' (the streams are then not kept); None: nothing follows."""
+        rows = streams.shape[0]
+        xb = self.rt.buffer("normed", self.dim)[:rows]
+        if start is not None:
+            ops.stream_mix(streams, start=start, read=self.mixer_read, gain=self.mixer_gain, eps=self.eps, out=xb)
+        y = self._result(self.mixer, rows)
+        self.mixer.forward(xb, y, batch, cache)
+        mix = self.mixer_mix
+        if self.feed_forward is not None:
+            ops.stream_mix(streams, result=y, mix=mix, read=self.ffn_read, gain=self.ffn_gain, eps=self.eps, out=xb)
+            y = self._result(self.feed_forward, rows)
+            self.feed_forward.forward(xb, y, batch)
+            mix = self.ffn_mix
+        if tail is None:
+            ops.stream_mix(streams, result=y, mix=mix)
+            return
+        read, gain, eps, out, picked = tail
+        ops.stream_mix(streams, result=y, mix=mix, read=read, gain=gain, eps=eps, out=out, row_index=picked, write=picked is None)
+
+
+register_block("hyper_connections", HyperConnectionBlock, replace=True)

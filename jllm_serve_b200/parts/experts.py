@@ -16,11 +16,15 @@ row does not use has weight 0 and adds exact zeros, as above. `shared`: a dense 
 every row runs, added to the same result.
 
 What a spec may ask of the router (`ops.route_experts`): `score` "softmax" (the scores are a softmax over all of the router's
-entries); `identity` entries behind the experts, chosen like experts, that have no weights and give the row's input itself
+entries); `router_bias` (a vector added to the entries' logits); `identity` entries behind the experts, chosen like experts, that have no weights and give the row's input itself
 times their weight (`ops.add_rows_scaled` with the sum of a row's chosen identity weights); `shared_gate`, a [1, dim] matrix
 whose logistic value per row multiplies the shared expert's result: its row rides behind the router's (one float32 matrix,
 one launch), and the shared expert rides behind the routed ones in both products as an expert that every row uses with that
 weight.
+
+With the clamped gated unit and weights on the output the first product's epilogue does all that is left to do (bfloat16): it cuts
+off (a shared expert's units at a limit of their own), gates, and multiplies by the row's weight (`ops.GluUnits`); where that epilogue
+does not take the sizes, and in float32, `ops.glu_clamped` does the same behind the product.
 """
 from __future__ import annotations
 
@@ -57,7 +61,7 @@ class RoutedExperts(FeedForward):
             downs.append(tensors.pop(prefix + "shared." + shared.names[2]))
         elif shared is not None and getattr(spec, "shared_gate", "") and shared.kind == "dense_glu" and shared.activation == spec.activation:
             # a gated shared expert (weights on the output): behind the routed ones in both products, its weight the row's gate
-            self.shared_ff = shared.hidden
+            self.shared_ff, self.shared_limit = shared.hidden, float(shared.limit)
             gates.append(tensors.pop(prefix + "shared." + shared.names[0]))
             ups.append(tensors.pop(prefix + "shared." + shared.names[1]))
             downs.append(tensors.pop(prefix + "shared." + shared.names[2]))
@@ -81,6 +85,11 @@ class RoutedExperts(FeedForward):
         del downs
         self.router = tensors.pop(prefix + "router")
         self.correction = tensors.pop(prefix + "correction") if spec.correction else None
+        self.router_bias = tensors.pop(prefix + spec.router_bias) if spec.router_bias else None
+        # the clamped unit with the weight on its result: what the first product's epilogue is told
+        self.clamped = spec.activation == "swish_clamped" and not self.on_input
+        self.words = tuple(ops.glu_descriptor("swish_clamped", limit) if self.clamped and limit else 0
+                           for limit in (float(spec.limit), self.shared_limit))
         self.identity = int(getattr(spec, "identity", 0))
         self.softmax = getattr(spec, "score", "sigmoid") == "softmax"
         self.gates = 0
@@ -96,6 +105,8 @@ class RoutedExperts(FeedForward):
         out = {prefix + "router": TensorWant((entries, dim), "matrix_fp32")}
         if spec.correction:
             out[prefix + "correction"] = TensorWant((entries,), "vector")
+        if getattr(spec, "router_bias", ""):
+            out[prefix + spec.router_bias] = TensorWant((entries,), "vector")
         if getattr(spec, "shared_gate", ""):
             out[prefix + spec.shared_gate] = TensorWant((1, dim), "matrix_fp32")
         for e in range(spec.experts):
@@ -110,12 +121,19 @@ class RoutedExperts(FeedForward):
         s, rows = self.spec, xb.shape[0]
         weights = self.rt.buffer("expert_weights", self.table, torch.float32)[:rows]
         ops.route_experts(xb, self.router, self.correction, s.top, s.scale * self.residual_scale, s.normalize, weights,
-                          identity=self.identity, gates=self.gates, softmax=self.softmax)
+                          identity=self.identity, gates=self.gates, softmax=self.softmax, bias=self.router_bias)
         h = self.rt.buffer("experts_hidden", self.hidden)[:rows]
         if self.on_input:
             gate_up = self.rt.buffer("experts_gate_up", 2 * self.hidden)[:rows]
             self.gate_up.forward(xb, gate_up)
             ops.glu_clamped(gate_up, weights, h, s.experts, s.hidden, s.limit, self.shared_ff, self.shared_limit)
+        elif self.clamped and self.fused:
+            units = ops.GluUnits(self.words[0], s.hidden, s.experts * s.hidden if self.shared_ff else 0, self.words[1], weights)
+            self.gate_up.forward(xb, h, swiglu=units)
+        elif self.clamped:
+            gate_up = self.rt.buffer("experts_gate_up", 2 * self.hidden)[:rows]
+            self.gate_up.forward(xb, gate_up)
+            ops.glu_clamped(gate_up, weights, h, s.experts, s.hidden, s.limit, self.shared_ff, self.shared_limit, on_output=True)
         else:
             if self.fused:
                 self.gate_up.forward(xb, h, swiglu=True)

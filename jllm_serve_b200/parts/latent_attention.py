@@ -18,6 +18,9 @@ What a spec may ask for beyond that (each on its own):
   q[:key_dim] . (Wuk c_j) + rot(q[key_dim:]) . r_j. A cached row is [c_j, r_j]; a head's latent-space query is [Wuk^T
   q[:key_dim], rot(q[key_dim:])], so the score is still ONE dot product with a cached row, and the attention runs with key and
   value heads of rank + rope_dim values: the last rope_dim values of its result are never read (Wuv takes the first rank).
+* `gate_full`: the gate has one value per value of the concatenated heads, applied in the same epilogue of the product with Wuv.
+* `tile_rows`: cached rows of `cache_dim` values, zeros behind the latent (a width the tile kernels take); the padded product
+  Wuk^T q makes the queries' zeros, and Wuv reads the first rank values of the result.
 * `own_latent` False: no down projection and no cache of its own; `cache` is another run's, whose rows it reads.
 """
 from __future__ import annotations
@@ -67,6 +70,12 @@ class LatentAttention(Mixer):
         self.q_up = Linear(tensors.pop(prefix + "uq")) if self.q_rank else None
         # Wuk [heads x dk, rank] as [heads, rank, dk]: the product that carries a head's query into the latent's space
         self.q_to_latent = tensors.pop(prefix + "uk").view(H, dk, R).transpose(1, 2).contiguous()
+        self.row = spec.cache_dim if self.plain else R + self.rope_dim       # values of a cached row
+        if self.plain and self.row != R:
+            filled = torch.zeros((H, self.row, dk), dtype=self.q_to_latent.dtype, device=self.q_to_latent.device)
+            filled[:, :R] = self.q_to_latent
+            self.q_to_latent = filled
+        self.gate_width = H * dv if spec.gate_full else H
         self.latent_to_v = tensors.pop(prefix + "uv").view(H, dv, R).contiguous()
         self.out = Linear(tensors.pop(prefix + "o"))
 
@@ -84,16 +93,16 @@ class LatentAttention(Mixer):
         if getattr(spec, "own_latent", True):
             out.update({prefix + "dkv": TensorWant((R + rd, dim)), prefix + "dkv.norm": TensorWant((R,), "vector", init="gain")})
         if spec.gated:
-            out[prefix + "g"] = TensorWant((H, dim))
+            out[prefix + "g"] = TensorWant((H * dv if getattr(spec, "gate_full", False) else H, dim))
         return out
 
     @classmethod
     def cache_need(cls, spec):
-        return PagedKeysValues(1, spec.rank + getattr(spec, "rope_dim", 0), spec.window, planes=1)
+        return PagedKeysValues(1, spec.cache_dim, spec.window, planes=1)
 
     def decode_bucket_cap(self, rows: int) -> int:
         s = self.spec
-        heads, width = min(s.heads, 16), s.rank + self.rope_dim
+        heads, width = min(s.heads, 16), self.row
         if not ops.attention_decode_fits(self.rt.dtype, heads, 1, width):
             return 1
         scratch = self.rt.buffer("attention_scratch", 2 << 20, torch.float32, rows=1)[0]
@@ -110,20 +119,21 @@ class LatentAttention(Mixer):
         if cache.writes:
             d_off = self.offsets["dkv"]
             ops.latent_norm_store(proj[:, d_off:d_off + R], self.latent_gain, s.norm_eps, batch.slots[cache.group], cache.keys)
-        q = self.rt.buffer("latent_queries", H * R)[:rows]
+        W = self.row
+        q = self.rt.buffer("latent_queries", H * W)[:rows]
         ops.gemm_heads(proj[:, :H * dk], self.q_to_latent, q)
-        att = self.rt.buffer("latent_attended", H * R)[:rows]
+        att = self.rt.buffer("latent_attended", H * W)[:rows]
         scratch = self.rt.buffer("attention_scratch", 2 << 20, torch.float32, rows=1)[0]
         # the decode kernel shares every key among at most 16 query heads: more heads go in groups of 16, each a launch
         # over the same cached rows
-        per = 16 if H > 16 and ops.attention_decode_fits(q.dtype, 16, 1, R) else H
+        per = 16 if H > 16 and ops.attention_decode_fits(q.dtype, 16, 1, W) else H
         for h0 in range(0, H, per):
             n = min(per, H - h0)
-            ops.attention(q[:, h0 * R:(h0 + n) * R], cache.keys, cache.values, att[:, h0 * R:(h0 + n) * R], batch,
-                          cache.group, n, 1, R, self.rt.page_size, s.window, s.scale, scratch)
+            ops.attention(q[:, h0 * W:(h0 + n) * W], cache.keys, cache.values, att[:, h0 * W:(h0 + n) * W], batch,
+                          cache.group, n, 1, W, self.rt.page_size, s.window, s.scale, scratch)
         y = self.rt.buffer("latent_values", H * dv)[:rows]
-        gate = proj[:, self.offsets["g"]:self.offsets["g"] + H] if s.gated else None
-        ops.gemm_heads(att, self.latent_to_v, y, gate, self.residual_scale)
+        gate = proj[:, self.offsets["g"]:self.offsets["g"] + self.gate_width] if s.gated else None
+        ops.gemm_heads(att, self.latent_to_v, y, gate, self.residual_scale, a_head=W)
         self.out.forward(y, x, accumulate=not self.overwrite)
 
     def _forward_general(self, xb, x, batch, cache) -> None:

@@ -45,7 +45,8 @@ class TensorWant:
     role: str = "matrix"                   # matrix | matrix_fp32 | vector | int_table
     optional: bool = False
     init: str = "normal"                   # random-weights mode: normal = N(0, 0.02), gain = 1 + N(0, 0.1),
-                                           # average = (1 + N(0, 0.1)) / the tensor's size
+                                           # average = (1 + N(0, 0.1)) / the tensor's size,
+                                           # identity = a square matrix near the identity
 
 
 def target_dtype(stored: torch.dtype, role: str, compute: torch.dtype) -> torch.dtype:

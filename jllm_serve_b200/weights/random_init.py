@@ -42,6 +42,8 @@ def random_tensors(wants: Dict[str, TensorWant], seed: int, device="cpu", dtype:
         t = torch.randn(want.shape, generator=gen, device=device, dtype=torch.float32)
         if want.init == "average":          # weights of a weighted mean: about 1 / n each
             t = (t * GAIN_STD + 1.0) / max(1, t.numel())
+        elif want.init == "identity":       # a square matrix near the identity
+            t = t * GAIN_STD + torch.eye(want.shape[0], device=device)
         else:
             t = t * GAIN_STD + 1.0 if want.init == "gain" else t * MATRIX_STD
         to = (vector_dtype or dtype) if want.role == "vector" else dtype
