@@ -13,7 +13,7 @@ read (every weight once plus the cache of the live requests) with the measured c
 `points` holds decode at batch 1 and 64; `check` compares the bfloat16 logits with the 32-bit path's at these
 layer sizes (two layers, untimed). Peaks come from MEASURED_PEAKS.json when it exists.
 
-`--design madevik`, `--design movivik`, `--design bozevik`, `--design guvolix` and `--design fusazen` are another program under the same roof and leave the default
+`--design madevik`, `--design movivik`, `--design bozevik`, `--design guvolix`, `--design fusazen` and `--design narolorn` are another program under the same roof and leave the default
 workload alone: prefill and decode of the Madevik design (gated linear attention, attention over a cached latent, routed
 experts), of the Movivik design (chunked and parallel attention layers, linear attention with fixed decays, norms in front of
 and behind every part) or of the Bozevik design (attention over a cached latent with a query latent and a shared rotated key
@@ -217,6 +217,22 @@ def fusazen_shape(width, heads, kv_heads, ff, runs, chunk=1024, vocab=32768):
             "embedding": {"scale": 2.0}, "layers": layers}
 
 
+def narolorn_shape(width, heads, kv_heads, rank, experts, top, ff, runs, span=1024, streams=4, vocab=32768):
+    """Layers in fours: two of attention over a cached latent under a window of `span` positions (a gate of full width), one whose values
+    are its keys (norms over all heads, rotation of every head, a chunk mask of `span` positions), one of capped scores over all
+    positions (queries that grow with the position); heads of 128 throughout; a residual of `streams` streams; routed experts with a
+    gated shared one in every layer."""
+    mlp = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "top": top}, "shared": {"ff": ff, "limit": 5.0}}
+    latent = {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": rank,
+                                                                "scale": 128 ** -0.5, "mask": {"size": span}}}
+    keys = {"type": "attention_2", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                                         "mask": {"size": span}, "rot": {"base": 10000.0, "dims": 128}}}
+    capped = {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128,
+                                                         "scale": 128 ** -0.5, "softcap": 30.0, "q_temp": {"coef": 0.1, "every": 512}}}
+    return {"architecture": "Narolorn", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "streams": streams, "logit_softcap": 30.0,
+            "layers": [(latent, latent, keys, capped)[i % 4] for i in range(runs)]}
+
+
 def movivik_parallel_shape(width, heads, kv_heads, ff, runs, vocab=32768):
     """A Movivik model of parallel layers only (the closest kin of the Guvolix shape): a causal attention beside linear
     attention with a fixed decay per head, heads of 128, a dense gated feed-forward."""
@@ -254,6 +270,12 @@ DESIGN_SIZES = {
                           movivik_shape(2048, 16, 8, 8192, 8), "movivik"),
                 "w4096": (fusazen_shape(4096, 32, 8, 18432, 4), _qwen3_shape(4096, 4, 32, 8, 12288),
                           movivik_shape(4096, 32, 8, 12288, 4), "movivik")},
+    # beside each the Qwen3 shape and a Bozevik model (latent attention with rows of the same width, clamped gated units, a shared
+    # expert in every second layer)
+    "narolorn": {"w2048": (narolorn_shape(2048, 16, 8, 256, 7, 2, 1024, 8), _qwen3_shape(2048, 8, 16, 8, 8192),
+                           bozevik_shape(2048, 16, 192, 64, 768, 7, 2, 1024, 8192, 8), "bozevik"),
+                 "w4096": (narolorn_shape(4096, 32, 8, 128, 15, 4, 768, 4), _qwen3_shape(4096, 4, 32, 8, 12288),
+                           bozevik_shape(4096, 32, 96, 32, 1536, 15, 4, 768, 12288, 4), "bozevik")},
 }
 
 
@@ -359,10 +381,10 @@ def _tensors_of(obj, seen=None):
 
 def main() -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawTextHelpFormatter)
-    ap.add_argument("--design", default="", choices=["", "madevik", "movivik", "bozevik", "guvolix", "fusazen"],
-                    help="madevik, movivik, bozevik, guvolix, fusazen: time that design beside the Qwen3 dense shape of equal size (bozevik: "
+    ap.add_argument("--design", default="", choices=["", "madevik", "movivik", "bozevik", "guvolix", "fusazen", "narolorn"],
+                    help="madevik, movivik, bozevik, guvolix, fusazen, narolorn: time that design beside the Qwen3 dense shape of equal size (bozevik: "
                          "also beside a Madevik model of latent-attention layers; guvolix: also beside a Movivik model of "
-                         "parallel layers; fusazen: also beside a Movivik model) instead of the default workload")
+                         "parallel layers; fusazen: also beside a Movivik model; narolorn: also beside a Bozevik model) instead of the default workload")
     ap.add_argument("--design-sizes", default="w2048,w4096", help="which of the sizes of --design, with commas between them")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=64)
