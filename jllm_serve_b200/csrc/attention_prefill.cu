@@ -55,7 +55,7 @@ __device__ __forceinline__ uint32_t tile_offset(int r, int c) {
     return (uint32_t)((r * (HD / 8) + (c ^ (r & 7))) * 16);
 }
 
-template <int HD>
+template <int HD, bool CAP>
 __global__ void __launch_bounds__(THREADS)
 attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ k_cache,
                          const __nv_bfloat16* __restrict__ v_cache, __nv_bfloat16* __restrict__ out, int out_stride,
@@ -180,13 +180,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
                 }
             }
             // ---- cap, mask and online softmax ----
-            const float to_log2 = cap ? 1.f : scale_log2;      // (a capped score is in base 2 already)
-            if (cap) {
-    #pragma unroll
-                for (int j = 0; j < BKV / 8; ++j)
-    #pragma unroll
-                    for (int i = 0; i < 4; ++i) s[j][i] = cap(s[j][i]);
-            }
+            const float to_log2 = CAP ? 1.f : scale_log2;      // (a capped score is in base 2 already)
+            if constexpr (CAP) cap.tile(reinterpret_cast<uint32_t(&)[BKV / 8][4]>(s));
             const int key0 = kt * BKV;
             float mx[2] = {-INFINITY, -INFINITY};
             // a tile that every row of this warp sees whole (all keys at or before the warp's first position and
@@ -284,7 +279,7 @@ int launch(const void* q, int q_stride, const void* k_cache, const void* v_cache
            int num_segs, int rows, int heads, int kv_heads, int page_size, int window, float scale,
            cudaStream_t stream, int keep_first, VecRef sink, float softcap) {
     const size_t smem = (size_t)BQ * HD * 2 + 4 * (size_t)BKV * HD * 2;
-    auto kern = attention_prefill_kernel<HD>;
+    auto kern = softcap > 0.f ? attention_prefill_kernel<HD, true> : attention_prefill_kernel<HD, false>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     const dim3 grid((rows + BQ - 1) / BQ + num_segs, heads);
     kern<<<grid, THREADS, smem, stream>>>((const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k_cache,

@@ -43,6 +43,7 @@ __device__ __forceinline__ void tcgen05_mma_bf16_ts(uint32_t tmem_d, uint32_t tm
         : "memory");
 }
 
+template <bool CAP>
 __global__ void __launch_bounds__(THREADS, 1)
 attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                               const __grid_constant__ CUtensorMap map_v, const __nv_bfloat16* __restrict__ k_cache,
@@ -229,7 +230,7 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
             const int P = pos0 + x * BQ + min(r, rows_x[x] - 1);   // rows past the end copy the last row, and are not stored
             const int lo = jllm_first_key(P, window);              // the first key this row sees (window or chunk)
             const int pos0_x = pos0 + x * BQ;
-            const float to_log2 = cap ? 1.f : scale_log2;          // (a capped score is in base 2 already)
+            const float to_log2 = CAP ? 1.f : scale_log2;          // (a capped score is in base 2 already)
             float m = -INFINITY, l = 0.f;
             bool ok = true;
             for (int j = 0; j < n_mine && ok; ++j) {
@@ -241,12 +242,7 @@ attention_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const _
 #pragma unroll
                 for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, v[c]);
                 tmem_ld_wait();
-                if (cap) {
-#pragma unroll
-                    for (int c = 0; c < 4; ++c)
-#pragma unroll
-                        for (int i = 0; i < 32; ++i) v[c][i] = __float_as_uint(cap(__uint_as_float(v[c][i])));
-                }
+                if constexpr (CAP) cap.tile(v);
                 if (masked) {
 #pragma unroll
                     for (int c = 0; c < 4; ++c)
@@ -376,7 +372,7 @@ JLLM_EXPORT int jllm_attention_prefill_pair(const void* q, int q_stride, const v
     if (!error_word) return jllm_fail(JLLM_CUDA_ERROR, "attention_prefill_pair: no error word");
     int page_shift = 0;
     while ((1 << page_shift) < page_size) ++page_shift;
-    auto kern = attention_prefill_pair_kernel;
+    auto kern = softcap > 0.f ? attention_prefill_pair_kernel<true> : attention_prefill_pair_kernel<false>;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
     const dim3 grid(heads, (rows + 2 * BQ - 1) / (2 * BQ) + num_segs);
     jllm_launch(kern, grid, dim3(THREADS), SMEM_BYTES, stream, true, map_q, map_k, map_v, (const __nv_bfloat16*)k_cache,

@@ -33,6 +33,7 @@ constexpr float LOG2E = 1.4426950408889634f;
 constexpr size_t SMEM_BYTES = 6 * TILE_BYTES + 1024 + 256;
 constexpr int TMEM_COLS = 512;                      // S0 at 0, S1 at 128, O at 256
 
+template <bool CAP>
 __global__ void __launch_bounds__(THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const __nv_bfloat16* __restrict__ k_cache,
@@ -212,7 +213,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const uint32_t lane_addr = tmem_base + ((uint32_t)(quad * 32) << 16);
         const int P = pos0 + min(r, rows_here - 1);            // rows past the end copy the last row, and are not stored
         const int lo = jllm_first_key(P, window);              // the first key this row sees (window or chunk)
-        const float to_log2 = cap ? 1.f : scale_log2;          // (a capped score is in base 2 already)
+        const float to_log2 = CAP ? 1.f : scale_log2;          // (a capped score is in base 2 already)
         float m = -INFINITY, l = 0.f;
         bool ok = true;
         for (int j = 0; j < n_tiles && ok; ++j) {
@@ -226,12 +227,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
             for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(lane_addr + b * 128 + c * 32, v[c]);
             tmem_ld_wait();
-            if (cap) {
-#pragma unroll
-                for (int c = 0; c < 4; ++c)
-#pragma unroll
-                    for (int i = 0; i < 32; ++i) v[c][i] = __float_as_uint(cap(__uint_as_float(v[c][i])));
-            }
+            if constexpr (CAP) cap.tile(v);
             if (masked) {
 #pragma unroll
                 for (int c = 0; c < 4; ++c)
@@ -398,7 +394,7 @@ static int prefill_tc_any(const void* q, int q_stride, const void* k_cache, cons
     if (!error_word) return jllm_fail(JLLM_CUDA_ERROR, "attention_prefill_tc: no error word");
     int page_shift = 0;
     while ((1 << page_shift) < page_size) ++page_shift;
-    auto kern = attention_prefill_tc_kernel;
+    auto kern = softcap > 0.f ? attention_prefill_tc_kernel<true> : attention_prefill_tc_kernel<false>;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
     const dim3 grid(heads, (rows + BQ - 1) / BQ + num_segs);
     jllm_launch(kern, grid, dim3(THREADS), SMEM_BYTES, stream, true, map_q, map_k, map_v, (const __nv_bfloat16*)k_cache,

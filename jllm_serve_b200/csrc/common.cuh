@@ -203,8 +203,8 @@ struct GluArgs {
     __device__ __forceinline__ float weight(int row, int unit) const {
         return weights[(size_t)row * ld_w + min((unit < split ? unit : split) / ff, ld_w - 1)];
     }
-    // whether eight units from a multiple of 8 on always share their word and their weight
-    __device__ __forceinline__ bool in_eights() const { return (ff & 7) == 0 && ((split & 7) == 0 || split == 0x7fffffff); }
+    // whether eight units from a multiple of 8 on always share their word and their weight (the products' epilogues count on it)
+    bool in_eights() const { return weights == nullptr && split == 0x7fffffff ? true : (ff & 7) == 0 && ((split & 7) == 0 || split == 0x7fffffff); }
     template <bool FAST>
     __device__ __forceinline__ float apply(float gate, float up, int row, int unit) const {
         const float y = glu_unit<FAST>(gate, up, word_of(unit));
@@ -231,11 +231,57 @@ __device__ __forceinline__ float unit_tanh(float x) {
     return 1.f - __fdividef(2.f, t + 1.f);
 }
 // What the bfloat16 attention kernels are told: a raw dot product d becomes the base-2 score out * tanh(in * d) with in =
-// scale / cap and out = cap * log2(e). out = 0: no cap.
+// scale / cap and out = cap * log2(e). out = 0: no cap. A prompt tile's scores go through `tile`: where none of a warp's values lies
+// beyond the cap (|x| <= 1 for x = in * d, nearly always) tanh is an odd polynomial of degree 13, two values at a time on the
+// multiply-add pipes (the special-function unit is what bounds these kernels' softmax); else `operator()`.
+// The polynomial interpolates tanh(x) / x at the seven Chebyshev points of x^2 in [0, 1]: within 1.2e-7 in float32.
 struct ScoreCap {
     float in, out;
     __host__ __device__ __forceinline__ explicit operator bool() const { return out != 0.f; }
     __device__ __forceinline__ float operator()(float d) const { return out * unit_tanh(in * d); }
+
+    __device__ static __forceinline__ uint64_t both(float v) {
+        uint64_t p;
+        asm("mov.b64 %0, {%1, %1};" : "=l"(p) : "f"(v));
+        return p;
+    }
+    // N x M raw products of a warp's threads, as the bits of floats; all threads of the warp call it
+    template <int N, int M>
+    __device__ __forceinline__ void tile(uint32_t (&v)[N][M]) const {
+        float far[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int c = 0; c < N; ++c)
+#pragma unroll
+            for (int i = 0; i < M; ++i) far[i & 3] = fmaxf(far[i & 3], fabsf(__uint_as_float(v[c][i])));
+        const float reach = fmaxf(fmaxf(far[0], far[1]), fmaxf(far[2], far[3])) * in;
+        if (__all_sync(0xffffffffu, reach <= 1.f)) {
+            const uint64_t c0 = both(out * 0.9999999403953552f), c1 = both(out * -0.3333282768726349f), c2 = both(out * 0.13325075805187225f),
+                           c3 = both(out * -0.053451646119356155f), c4 = both(out * 0.02027970738708973f),
+                           c5 = both(out * -0.0061943246982991695f), c6 = both(out * 0.0010380251333117485f), k = both(in);
+#pragma unroll
+            for (int c = 0; c < N; ++c)
+#pragma unroll
+                for (int i = 0; i < M; i += 2) {
+                    uint64_t x, t, q;
+                    asm("mov.b64 %0, {%1, %2};" : "=l"(x) : "r"(v[c][i]), "r"(v[c][i + 1]));
+                    asm("mul.rn.f32x2 %0, %0, %1;" : "+l"(x) : "l"(k));
+                    asm("mul.rn.f32x2 %0, %1, %1;" : "=l"(t) : "l"(x));
+                    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(q) : "l"(c6), "l"(t), "l"(c5));
+                    asm("fma.rn.f32x2 %0, %0, %1, %2;" : "+l"(q) : "l"(t), "l"(c4));
+                    asm("fma.rn.f32x2 %0, %0, %1, %2;" : "+l"(q) : "l"(t), "l"(c3));
+                    asm("fma.rn.f32x2 %0, %0, %1, %2;" : "+l"(q) : "l"(t), "l"(c2));
+                    asm("fma.rn.f32x2 %0, %0, %1, %2;" : "+l"(q) : "l"(t), "l"(c1));
+                    asm("fma.rn.f32x2 %0, %0, %1, %2;" : "+l"(q) : "l"(t), "l"(c0));
+                    asm("mul.rn.f32x2 %0, %0, %1;" : "+l"(q) : "l"(x));
+                    asm("mov.b64 {%0, %1}, %2;" : "=r"(v[c][i]), "=r"(v[c][i + 1]) : "l"(q));
+                }
+        } else {
+#pragma unroll
+            for (int c = 0; c < N; ++c)
+#pragma unroll
+                for (int i = 0; i < M; ++i) v[c][i] = __float_as_uint((*this)(__uint_as_float(v[c][i])));
+        }
+    }
 };
 inline ScoreCap score_cap(float cap, float scale) { return cap > 0.f ? ScoreCap{scale / cap, cap * 1.4426950408889634f} : ScoreCap{0.f, 0.f}; }
 

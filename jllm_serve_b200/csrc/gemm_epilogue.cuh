@@ -112,19 +112,14 @@ struct TileEpilogue {
             Tout* dst = out + (size_t)row * ldo + (n_base >> 1);
             // (the tensor-core path may use the fast exponential: its result is rounded to bfloat16 anyway)
             float hv[16];
-            const int unit0 = n_base >> 1;
-            const bool weighted = swiglu.weights != nullptr, eights = swiglu.in_eights();
-            float wt[2] = {1.f, 1.f};
-            if (weighted && eights) {
-                wt[0] = swiglu.weight(row, unit0);
-                wt[1] = swiglu.weight(row, unit0 + 8);
-            }
+            // (eight neighbouring units share their word and their weight: the launchers see to it)
 #pragma unroll
-            for (int j = 0; j < 16; ++j) {
-                const int cg = (j >> 3) * 16 + (j & 7);
-                const float gt = __uint_as_float(v[cg]), up = __uint_as_float(v[cg + 8]);
-                hv[j] = glu_unit<true>(gt, up, swiglu.word_of(unit0 + j));
-                if (weighted) hv[j] = __fmul_rn(hv[j], eights ? wt[j >> 3] : swiglu.weight(row, unit0 + j));
+            for (int b = 0; b < 2; ++b) {
+                const int unit = (n_base >> 1) + 8 * b, word = swiglu.word_of(unit);
+                const float wt = swiglu.weights != nullptr ? swiglu.weight(row, unit) : 1.f;
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                    hv[8 * b + j] = __fmul_rn(glu_unit<true>(__uint_as_float(v[16 * b + j]), __uint_as_float(v[16 * b + j + 8]), word), wt);
             }
             if (sizeof(Tout) == 2 && n_base + 32 <= N && ((((uintptr_t)dst) & 15u) == 0)) {
                 uint32_t p[8];

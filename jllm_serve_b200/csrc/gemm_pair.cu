@@ -476,6 +476,7 @@ JLLM_EXPORT int jllm_gemm_pair(const void* a, int lda, const void* w, int k_bloc
                                int swiglu_word, const void* glu_more, float* workspace, long long workspace_floats, int stream_mode,
                                cudaStream_t stream) {
     const GluArgs swiglu = glu_args(swiglu_word, glu_more);
+    JLLM_REQUIRE(swiglu.in_eights(), "gemm_pair: units of %d in front of %d do not come in eights", swiglu.ff, swiglu.split);
     JLLM_REQUIRE(jllm_gemm_pair_fits(a, lda, w, M, N, K),
                  "gemm_pair: needs K %% 8 == 0 and 16-byte aligned rows (M=%d N=%d K=%d lda=%d)", M, N, K, lda);
     JLLM_REQUIRE(k_blocks_packed == (K + BK - 1) / BK, "gemm_pair: the packed weight has %d k blocks, K=%d needs %d",

@@ -211,6 +211,7 @@ JLLM_EXPORT int jllm_gemm_small_m(const void* a, int lda, const void* w, int k_b
                                   void* out, int out_dtype, int ldo, int accumulate, int M, int N, int K,
                                   int swiglu_word, const void* glu_more, cudaStream_t stream) {
     const GluArgs swiglu = glu_args(swiglu_word, glu_more);
+    JLLM_REQUIRE(swiglu.in_eights(), "gemm_small_m: units of %d in front of %d do not come in eights", swiglu.ff, swiglu.split);
     JLLM_REQUIRE(jllm_gemm_small_m_fits(a, lda, w, M, N, K),
                  "gemm_small_m: needs 1 <= M <= 64, K %% 8 == 0 and 16-byte aligned rows (M=%d N=%d K=%d lda=%d)",
                  M, N, K, lda);

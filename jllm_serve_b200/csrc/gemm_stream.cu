@@ -328,6 +328,7 @@ JLLM_EXPORT int jllm_gemm_stream(const void* a, int lda, const void* w_packed, i
                                  int swiglu_word, const void* glu_more, float* workspace, long long workspace_floats, int max_blocks,
                                  cudaStream_t stream) {
     const GluArgs swiglu = glu_args(swiglu_word, glu_more);
+    JLLM_REQUIRE(swiglu.in_eights(), "gemm_stream: units of %d in front of %d do not come in eights", swiglu.ff, swiglu.split);
     JLLM_REQUIRE(M >= 1 && M <= MAX_TOKENS && N >= 1 && K >= 8 && K % 8 == 0 && lda % 8 == 0 && ((uintptr_t)a % 16) == 0 &&
                      ((uintptr_t)w_packed % 16) == 0,
                  "gemm_stream: needs 1 <= rows <= %d, K %% 8 == 0 and 16-byte aligned rows and weights "

@@ -375,6 +375,7 @@ JLLM_EXPORT int jllm_gemm_tcgen05(const void* a, int lda, const void* w, int k_b
                                   int swiglu_word, const void* glu_more, float* workspace, long long workspace_floats, int stream_mode,
                                   int tile_width, cudaStream_t stream) {
     const GluArgs swiglu = glu_args(swiglu_word, glu_more);
+    JLLM_REQUIRE(swiglu.in_eights(), "gemm_tcgen05: units of %d in front of %d do not come in eights", swiglu.ff, swiglu.split);
     JLLM_REQUIRE(jllm_gemm_tcgen05_fits(a, lda, w, M, N, K),
                  "gemm_tcgen05: needs K %% 8 == 0 and 16-byte aligned rows (M=%d N=%d K=%d lda=%d)", M, N, K, lda);
     JLLM_REQUIRE(k_blocks_packed == (K + BK - 1) / BK, "gemm_tcgen05: the packed weight has %d k blocks, K=%d needs %d",

@@ -662,7 +662,7 @@ class _GluMore(ctypes.Structure):          # (GluMore in common.cuh)
 class GluUnits:
     """A product's `swiglu` argument where the stacked units are several feed-forwards': units from `split` on (0: none) have an
     activation word of their own, and with `weights` ([rows, columns] float32) unit u's result is multiplied by weights[row, u // ff],
-    a unit's from `split` on by weights[row, split // ff]."""
+    a unit's from `split` on by weights[row, split // ff]. ff and split are multiples of 8."""
 
     def __init__(self, word: int, ff: int, split: int = 0, word_behind: int = 0, weights: torch.Tensor | None = None):
         assert weights is None or (weights.dtype == torch.float32 and weights.stride(1) == 1)

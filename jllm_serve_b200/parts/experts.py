@@ -74,6 +74,8 @@ class RoutedExperts(FeedForward):
         del gates, ups
         # (a weight in front of the gated unit rules out the product's own epilogue, which gates what it has summed)
         self.fused = gate.dtype == torch.bfloat16 and dim % 8 == 0 and self.hidden % 8 == 0 and not self.on_input
+        if spec.activation == "swish_clamped" and ff % 8:        # (the epilogue takes limits and weights for eight units at a time)
+            self.fused = False
         if self.fused:      # blocks of 8 gate rows followed by their 8 up rows: the product's epilogue applies SwiGLU
             stacked = torch.stack([gate.view(self.hidden // 8, 8, dim), up.view(self.hidden // 8, 8, dim)], dim=1)
             self.gate_up = Linear(stacked.reshape(2 * self.hidden, dim).contiguous())
