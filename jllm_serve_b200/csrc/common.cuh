@@ -111,6 +111,14 @@ __device__ __forceinline__ long long jllm_page_of(const int* __restrict__ table,
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void pdl_trigger() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 
+// Weights are nobody's output: a kernel may ask for its own before it waits for its predecessor. `bytes` from `p` on, whole lines,
+// asked of memory by the block's threads together.
+__device__ __forceinline__ void prefetch_lines(const void* p, size_t bytes) {
+    const char* c = static_cast<const char*>(p);
+    for (size_t i = (size_t)threadIdx.x * 128; i < bytes; i += (size_t)blockDim.x * 128)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(c + i));
+}
+
 bool jllm_pdl_enabled();
 enum : int { LAUNCH_PLAIN = 0, LAUNCH_DEPENDENT = 1, LAUNCH_DEPENDENT_WANTS_L1 = 2 };
 bool jllm_launch_overlaps(size_t dynamic_smem, int how);     // decides, and keeps the record the decision needs

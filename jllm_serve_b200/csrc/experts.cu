@@ -28,6 +28,11 @@ route_experts_kernel(const T* __restrict__ h, int ld, const float* __restrict__ 
     float* s = smem;                   // [experts] scores
     float* c = s + (experts + 1) / 2 * 2;      // [experts] choice scores, -inf once taken
     float* hs = c + (experts + 1) / 2 * 2;     // [dim] the row, read once (on a 16-byte boundary)
+    if (blockIdx.x < 8) {              // the router matrix comes from memory while the kernel in front still runs: a part per block
+        const size_t all = (size_t)experts * dim * sizeof(float), parts = min(8u, gridDim.x), part = ((all + parts - 1) / parts + 127) & ~(size_t)127;
+        const size_t from = min(all, blockIdx.x * part);
+        prefetch_lines(reinterpret_cast<const char*>(router) + from, min(part, all - from));
+    }
     pdl_wait();
     pdl_trigger();
     const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;

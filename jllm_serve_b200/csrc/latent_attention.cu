@@ -239,6 +239,8 @@ gemm_heads_mma_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_b
                       int gate_full, float alpha, int M, int N, int K, int a_head, int o_head, HeadRope rp) {
     __shared__ __align__(16) __nv_bfloat16 as[64][HPAD];
     __shared__ __align__(16) __nv_bfloat16 ws[64][HPAD];
+    if (blockIdx.y == 0 && (int)blockIdx.x * 64 < N)       // (the block's weight rows come from memory while the kernel in front still runs)
+        prefetch_lines(w + ((size_t)blockIdx.z * N + blockIdx.x * 64) * K, (size_t)min(64, N - (int)blockIdx.x * 64) * K * 2);
     pdl_wait();
     pdl_trigger();
     if (rp.rope_dim > 0 && blockIdx.x == gridDim.x - 1) {

@@ -48,6 +48,13 @@ stream_mix_kernel(float* __restrict__ X, const float* __restrict__ x0, const flo
                 v[s][k] = i < groups ? xr[(size_t)s * groups + i] : zero;
             }
     }
+    // (so are the weights, which nobody writes)
+    float m[S * S + S], in[S];
+#pragma unroll
+    for (int j = 0; j < S * S + S; ++j) m[j] = coef != nullptr ? __ldg(coef + j) : 0.f;
+#pragma unroll
+    for (int j = 0; j < S; ++j) in[j] = read != nullptr ? __ldg(read + j) : 0.f;
+    if (read != nullptr && r < 8) prefetch_lines(gain.p, (size_t)dim * (gain.dtype == JLLM_F32 ? 4 : 2));
     pdl_wait();
     pdl_trigger();
     if (x0 != nullptr) {
@@ -68,9 +75,6 @@ stream_mix_kernel(float* __restrict__ X, const float* __restrict__ x0, const flo
             const int i = threadIdx.x + k * blockDim.x;
             yv[k] = i < groups ? yr[i] : zero;
         }
-        float m[S * S + S];
-#pragma unroll
-        for (int j = 0; j < S * S + S; ++j) m[j] = __ldg(coef + j);
 #pragma unroll
         for (int k = 0; k < N; ++k) {
             float4 n[S];
@@ -99,9 +103,9 @@ stream_mix_kernel(float* __restrict__ X, const float* __restrict__ x0, const flo
     float ss = 0.f;
 #pragma unroll
     for (int k = 0; k < N; ++k) {
-        u[k] = scaled4(__ldg(read), v[0][k]);
+        u[k] = scaled4(in[0], v[0][k]);
 #pragma unroll
-        for (int s = 1; s < S; ++s) add_scaled4(u[k], __ldg(read + s), v[s][k]);
+        for (int s = 1; s < S; ++s) add_scaled4(u[k], in[s], v[s][k]);
         ss = fmaf(u[k].x, u[k].x, fmaf(u[k].y, u[k].y, fmaf(u[k].z, u[k].z, fmaf(u[k].w, u[k].w, ss))));
     }
     ss = block_sum(ss, scratch);
