@@ -145,6 +145,129 @@ map_prepare_kernel(const T* __restrict__ src, MapShape s, const float* __restric
     }
 }
 
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+__device__ __forceinline__ float4 gained4(float4 v, float f, float4 g) {
+    return make_float4(__fmul_rn(__fmul_rn(v.x, f), g.x), __fmul_rn(__fmul_rn(v.y, f), g.y), __fmul_rn(__fmul_rn(v.z, f), g.z),
+                       __fmul_rn(__fmul_rn(v.w, f), g.w));
+}
+
+// The same for rows that are normed and rotated by halves (or not at all), where every piece is whole and aligned: the row's queries
+// and keys are read once, into shared memory as float32, both sums of squares meet in one reduction, and a thread turns both pieces of
+// a pair, so a gain and an angle are read once. Four values a thread at a time: neighbouring threads then read neighbouring 16 bytes.
+template <typename T>
+__global__ void __launch_bounds__(256)
+map_prepare_normed_kernel(const T* __restrict__ src, MapShape s, const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps,
+                          const float* __restrict__ cos_t, const float* __restrict__ sin_t, const int* __restrict__ positions,
+                          const int* __restrict__ slots, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
+                          int write_kv, int num_slots) {
+    extern __shared__ __align__(16) float staged[];        // the query columns, then the key columns
+    __shared__ float sums[2][8];
+    const size_t r = blockIdx.x;
+    const int q_cols = s.heads * s.maps * s.dim, k_cols = write_kv ? s.kv_heads * s.maps * s.dim : 0, tid = threadIdx.x;
+    // (positions and slots came from the host before the step)
+    const int pos = positions[r], slot = write_kv ? slots[r] : 0, half = s.rotary_dim >> 1, W = s.width;
+    const float* cs = s.rotary_dim ? cos_t + (size_t)pos * half : nullptr;
+    const float* sn = s.rotary_dim ? sin_t + (size_t)pos * half : nullptr;
+    const float temp = s.temp_every > 0 ? fmaf(s.temp_coef, logf((float)((pos + 1) / s.temp_every + 1)), 1.f) : 1.f;
+    pdl_wait();
+    pdl_trigger();
+    const T* row = src + r * s.ld;
+    float ss[2] = {0.f, 0.f};
+    for (int i = tid * 4; i < q_cols + k_cols; i += 1024) {
+        const float4 v = load4(i < q_cols ? row + i : row + s.k_off + (i - q_cols));
+        const float a = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+        if (i < q_cols) ss[0] += a;
+        else ss[1] += a;
+        store4(staged + i, v);
+    }
+#pragma unroll
+    for (int w = 0; w < 2; ++w) {
+        const float part = warp_sum(ss[w]);
+        if ((tid & 31) == 0) sums[w][tid >> 5] = part;
+    }
+    __syncthreads();
+    float inv[2];
+#pragma unroll
+    for (int w = 0; w < 2; ++w) {
+        float all = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) all += sums[w][i];
+        inv[w] = 1.f / sqrtf(all / (float)max(1, w == 0 ? q_cols : k_cols) + eps);
+    }
+    // both pieces of the pair at place i < half of the map whose columns begin at `col` of `part`, times f, to dst and dst + half
+    auto turn = [&](const float* part, const float* gain, float f, int col, int i, float t, T* dst) {
+        const float4 u = gained4(load4(part + col + i), f, load4(gain + col + i));
+        const float4 w = gained4(load4(part + col + half + i), f, load4(gain + col + half + i));
+        const float4 c = load4(cs + i), d = load4(sn + i);
+        float4 a, b;
+        a.x = __fmaf_rn(u.x, c.x, -__fmul_rn(w.x, d.x)); b.x = __fmaf_rn(w.x, c.x, __fmul_rn(u.x, d.x));
+        a.y = __fmaf_rn(u.y, c.y, -__fmul_rn(w.y, d.y)); b.y = __fmaf_rn(w.y, c.y, __fmul_rn(u.y, d.y));
+        a.z = __fmaf_rn(u.z, c.z, -__fmul_rn(w.z, d.z)); b.z = __fmaf_rn(w.z, c.z, __fmul_rn(u.z, d.z));
+        a.w = __fmaf_rn(u.w, c.w, -__fmul_rn(w.w, d.w)); b.w = __fmaf_rn(w.w, c.w, __fmul_rn(u.w, d.w));
+        if (t != 1.f) {
+            a = make_float4(__fmul_rn(a.x, t), __fmul_rn(a.y, t), __fmul_rn(a.z, t), __fmul_rn(a.w, t));
+            b = make_float4(__fmul_rn(b.x, t), __fmul_rn(b.y, t), __fmul_rn(b.z, t), __fmul_rn(b.w, t));
+        }
+        store4(dst + i, a);
+        store4(dst + half + i, b);
+    };
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const int pairs = half >> 2, q_items = pairs + ((W - s.rotary_dim) >> 2);
+    for (int e = tid; e < s.heads * s.maps * q_items; e += 256) {
+        const int hm = e / q_items, j = e - hm * q_items, at = (hm % s.maps) * s.dim;        // (the map's place in its row of W values)
+        T* dst = q_out + r * s.ld_q + (size_t)hm * W;
+        if (j < pairs) {
+            turn(staged, q_gain, inv[0], hm * s.dim, j * 4, temp, dst + at);
+        } else {
+            int p = (j - pairs) * 4;
+            if (p >= at) p += s.rotary_dim;
+            const int i = p - at;
+            float4 v = zero;
+            if (i >= 0 && i < s.dim) {
+                v = gained4(load4(staged + hm * s.dim + i), inv[0], load4(q_gain + hm * s.dim + i));
+                if (temp != 1.f) v = make_float4(__fmul_rn(v.x, temp), __fmul_rn(v.y, temp), __fmul_rn(v.z, temp), __fmul_rn(v.w, temp));
+            }
+            store4(dst + p, v);
+        }
+    }
+    if (!write_kv || !jllm_in_bounds(slot, num_slots, BOUNDS_SLOT)) return;
+    const size_t page = slot / s.page_size, off = slot % s.page_size;
+    const float* keys = staged + q_cols;
+    const int kv_items = s.maps * pairs + ((W - s.maps * s.rotary_dim) >> 2), plain = s.dim - s.rotary_dim;
+    for (int e = tid; e < s.kv_heads * kv_items; e += 256) {
+        const int g = e / kv_items, j = e - g * kv_items;
+        T* dst = k_cache + ((page * s.kv_heads + g) * s.page_size + off) * W;
+        if (j < s.maps * pairs) {
+            const int m = j / pairs;
+            turn(keys, k_gain, inv[1], (g * s.maps + m) * s.dim, (j - m * pairs) * 4, 1.f, dst + m * s.dim);
+        } else {
+            const int p = (j - s.maps * pairs) * 4, m = plain > 0 ? p / plain : s.maps;
+            if (m < s.maps) {
+                const int i = s.rotary_dim + p - m * plain, col = (g * s.maps + m) * s.dim + i;
+                store4(dst + m * s.dim + i, gained4(load4(keys + col), inv[1], load4(k_gain + col)));
+            } else {
+                store4(dst + s.maps * s.rotary_dim + p, zero);
+            }
+        }
+    }
+    const bool own = s.v_off == s.k_off;                   // the values are the keys as projected
+    for (int e = tid * 4; e < s.kv_heads * W; e += 1024) {
+        const int g = e / W, cc = e - g * W;
+        const float4 v = cc >= s.vdim ? zero : own ? load4(keys + g * s.vdim + cc) : load4(row + s.v_off + (size_t)g * s.vdim + cc);
+        store4(v_cache + ((page * s.kv_heads + g) * s.page_size + off) * W + cc, v);
+    }
+}
+
 // One warp per (row, head); V values a lane at a time.
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
@@ -224,6 +347,18 @@ JLLM_EXPORT int jllm_map_prepare(const void* src, int dtype, int ld, int k_off, 
     const bool vec = whole(dim) && whole(vdim) && whole(width) && whole(ld) && whole(k_off) && whole(v_off) && whole(ld_q) &&
                      whole(rotary_dim) && whole(rotary_dim / 2) &&
                      (((uintptr_t)src | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) % 16) == 0;
+    const size_t staged_bytes = ((size_t)heads * maps * dim + (size_t)kv_heads * maps * dim) * sizeof(float);
+    const bool gains_whole = (((uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)cos_t | (uintptr_t)sin_t) % 16) == 0;
+    if (vec && gains_whole && q_gain != nullptr && (k_gain != nullptr || !write_kv) && staged_bytes <= 46 * 1024 &&
+        (pairing == 0 || rotary_dim == 0)) {
+#define JLLM_MAP_NORMED(T)                                                                                                       \
+    jllm_launch(map_prepare_normed_kernel<T>, dim3(rows), dim3(256), staged_bytes, stream, LAUNCH_DEPENDENT, (const T*)src, s, q_gain, k_gain, \
+                eps, cos_t, sin_t, positions, slots, (T*)q_out, (T*)k_cache, (T*)v_cache, write_kv, num_slots)
+        if (dtype == JLLM_F32) JLLM_MAP_NORMED(float);
+        else JLLM_MAP_NORMED(__nv_bfloat16);
+#undef JLLM_MAP_NORMED
+        return jllm_check_launch("map_prepare");
+    }
 #define JLLM_MAP_PREPARE(T, N)                                                                                                 \
     jllm_launch(map_prepare_kernel<T, N>, dim3(rows), dim3(256), 0, stream, LAUNCH_DEPENDENT, (const T*)src, s, q_gain, k_gain, eps, cos_t, \
                 sin_t, positions, slots, (T*)q_out, (T*)k_cache, (T*)v_cache, write_kv, num_slots)

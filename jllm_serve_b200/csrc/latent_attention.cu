@@ -233,13 +233,13 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint3
 }
 
 template <bool VEC>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, VEC ? 7 : 5)      // (72 registers: 2,048 blocks of a prompt are two rounds of seven to an SM)
 gemm_heads_mma_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfloat16* __restrict__ w,
                       __nv_bfloat16* __restrict__ out, int ldo, const __nv_bfloat16* __restrict__ gate, int ld_gate,
                       int gate_full, float alpha, int M, int N, int K, int a_head, int o_head, HeadRope rp) {
     __shared__ __align__(16) __nv_bfloat16 as[64][HPAD];
     __shared__ __align__(16) __nv_bfloat16 ws[64][HPAD];
-    if (blockIdx.y == 0 && (int)blockIdx.x * 64 < N)       // (the block's weight rows come from memory while the kernel in front still runs)
+    if (gridDim.y == 1 && (int)blockIdx.x * 64 < N)        // (few rows: the block's weight rows come from memory while the kernel in front still runs)
         prefetch_lines(w + ((size_t)blockIdx.z * N + blockIdx.x * 64) * K, (size_t)min(64, N - (int)blockIdx.x * 64) * K * 2);
     pdl_wait();
     pdl_trigger();

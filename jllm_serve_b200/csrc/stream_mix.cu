@@ -45,7 +45,7 @@ stream_mix_kernel(float* __restrict__ X, const float* __restrict__ x0, const flo
 #pragma unroll
             for (int k = 0; k < N; ++k) {
                 const int i = threadIdx.x + k * blockDim.x;
-                v[s][k] = i < groups ? xr[(size_t)s * groups + i] : zero;
+                v[s][k] = i < groups ? __ldcg(xr + (size_t)s * groups + i) : zero;
             }
     }
     // (so are the weights, which nobody writes)
