@@ -20,7 +20,8 @@ and behind every part) or of the Bozevik design (attention over a cached latent 
 part, layer norms behind the parts, token shift, depth mix, clamped gated units) or of the Guvolix design (one norm per
 layer that feeds an attention with a sink and kept first tokens beside a selective state space or a matrix memory, and a
 dense or routed feed-forward) or of the Fusazen design (a delta rule, differential attention, attention with norms over all
-heads, a convolution over every mixer's input) at layer sizes that resemble a real model's, beside the Qwen3 dense shape of the same width, heads, layers and feed-forward weights (`--design-sizes`
+heads, a convolution over every mixer's input) or of the Narolorn design (a residual of several streams, capped attention, latent
+attention under a window, keys as values, routed clamped units) at layer sizes that resemble a real model's, beside the Qwen3 dense shape of the same width, heads, layers and feed-forward weights (`--design-sizes`
 picks among them); one JSON line with both models' figures per size.
 
 The engine runs on one GPU; for --gpus above 1 the program says so and exits with 2.

@@ -293,6 +293,26 @@ struct ScoreCap {
 };
 inline ScoreCap score_cap(float cap, float scale) { return cap > 0.f ? ScoreCap{scale / cap, cap * 1.4426950408889634f} : ScoreCap{0.f, 0.f}; }
 
+// N gated units whose activation is one word's, as a product's epilogue has them: the activation is chosen ONCE, in front of the loop
+// (a choice per unit makes a chain of branches of it, and a thread's units wait for one another).
+template <int N, typename Gate, typename Up>
+__device__ __forceinline__ void glu_units(int word, Gate gate, Up up, float factor, float (&out)[N]) {
+    if ((word & 3) == GLU_SWISH_CLAMPED) {
+        const float limit = __int_as_float(word & ~3);
+#pragma unroll
+        for (int j = 0; j < N; ++j) {
+            const float g = fminf(gate(j), limit), u = fminf(fmaxf(up(j), -limit), limit);
+            out[j] = __fmul_rn(__fdividef(g, 1.f + __expf(-kSwishAlpha * g)) * (u + 1.f), factor);
+        }
+    } else if (word == GLU_GELU_TANH) {
+#pragma unroll
+        for (int j = 0; j < N; ++j) out[j] = __fmul_rn(__fmul_rn(glu_act<true>(gate(j), GLU_GELU_TANH), up(j)), factor);
+    } else {
+#pragma unroll
+        for (int j = 0; j < N; ++j) out[j] = __fmul_rn(__fmul_rn(glu_act<true>(gate(j), GLU_SILU), up(j)), factor);
+    }
+}
+
 // What a product does with its result, the launchers' `accumulate` argument: 0 store it, 1 add it to what `out` holds, 2
 // store max(v, 0)^2 (the activation of an ungated feed-forward; behind the bias).
 enum : int { EPI_STORE = 0, EPI_ADD = 1, EPI_RELU2 = 2 };

@@ -117,9 +117,11 @@ struct TileEpilogue {
             for (int b = 0; b < 2; ++b) {
                 const int unit = (n_base >> 1) + 8 * b, word = swiglu.word_of(unit);
                 const float wt = swiglu.weights != nullptr ? swiglu.weight(row, unit) : 1.f;
+                float eight[8];
+                glu_units<8>(word, [&](int j) { return __uint_as_float(v[16 * b + j]); }, [&](int j) { return __uint_as_float(v[16 * b + j + 8]); },
+                             wt, eight);
 #pragma unroll
-                for (int j = 0; j < 8; ++j)
-                    hv[8 * b + j] = __fmul_rn(glu_unit<true>(__uint_as_float(v[16 * b + j]), __uint_as_float(v[16 * b + j + 8]), word), wt);
+                for (int j = 0; j < 8; ++j) hv[8 * b + j] = eight[j];
             }
             if (sizeof(Tout) == 2 && n_base + 32 <= N && ((((uintptr_t)dst) & 15u) == 0)) {
                 uint32_t p[8];

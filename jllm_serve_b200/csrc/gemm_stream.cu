@@ -180,12 +180,16 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_a, const __nv_bfloat1
                 if (swiglu) {
                     // rows come in blocks of 16: 8 gate rows, then the 8 up rows of the same hidden units
                     const int unit = (n >> 4) * 8 + (n & 7);
+                    float other[16], units[16];
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) {
-                        const float other = __shfl_xor_sync(0xffffffffu, v[j], 8);
-                        if ((lane & 8) == 0 && n + 8 < N && m0 + j < M) {
-                            const float gt = v[j];
-                            out[(size_t)(m0 + j) * ldo + unit] = from_float<Tout>(swiglu.apply<true>(gt, other, m0 + j, unit));
+                    for (int j = 0; j < 16; ++j) other[j] = __shfl_xor_sync(0xffffffffu, v[j], 8);
+                    if ((lane & 8) == 0 && n + 8 < N) {
+                        glu_units<16>(swiglu.word_of(unit), [&](int j) { return v[j]; }, [&](int j) { return other[j]; }, 1.f, units);
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) {
+                            if (m0 + j >= M) continue;
+                            if (swiglu.weights != nullptr) units[j] = __fmul_rn(units[j], swiglu.weight(m0 + j, unit));
+                            out[(size_t)(m0 + j) * ldo + unit] = from_float<Tout>(units[j]);
                         }
                     }
                 } else if (n < N) {
